@@ -62,13 +62,15 @@ class LayerCall:
     ``cache`` is the cache this call's mixer works on.  A call that does not own its cache
     (``writes_cache=False``) reads what an earlier call with the same ``cache`` id stored.
     ``before`` names an entry of ``ModelSpec.stream_parts`` that transforms the stream right
-    before this call's layer runs (None: nothing).
+    before this call's layer runs (None: nothing); ``turn`` is the number of the run of a repeated
+    stretch that starts here, for a stream part that asks for it (``wants_turn``).
     """
 
     layer: int
     cache: int
     writes_cache: bool = True
     before: Optional[int] = None
+    turn: int = 0
 
 
 @dataclass(frozen=True)

@@ -1,7 +1,7 @@
-// The gated delta rule with a decay per key channel: a recurrent mixer whose state is a matrix S [dim, vdim] per head.
+// The gated delta rule with a decay per key channel or per head: a recurrent mixer whose state is a matrix S [dim, vdim] per head.
 //
 // Per token and head, with unit vectors q (times dim^-1/2) and k, a value v, a write strength beta in (0, 1) and a decay
-// g in (0, 1) per key channel:
+// g in (0, 1) per key channel (or one for the whole head: HEAD below):
 //     S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
 // q, k and v come out of a short causal convolution over time (one filter per channel, the last tap is the current
 // token's) followed by silu; the convolution's last `taps - 1` inputs are part of the state.
@@ -18,6 +18,8 @@
 //   delta_scan   the recurrence over a step's tokens of every sequence; the tokens' vectors come through two stages of
 //                shared memory filled by cp.async a chunk ahead; the CTAs of a sequence also move the convolution's tail
 //                on, a share of the channels each.
+// With ONE decay per head the two dot products are taken from the column as it is and multiplied by the decay behind the
+// reduction (g (k . s_j) = k . (g s_j)), so the multiplication of the column leaves the chain from token to token.
 // State of a slot (float32): S as [heads, vdim, dim] (a column is contiguous), then the tail [taps - 1, channels].
 #include "common.cuh"
 
@@ -29,7 +31,9 @@ __device__ __forceinline__ float softplus_f32(float z) { return z > 20.0f ? z : 
 constexpr int kMaxTaps = 8;
 
 // proj rows: [.. q (G * D) | k (G * D) | v (H * V) .. | b (H) ..] at col_off / b_off, row stride ld, activation type A.
-// z: float32 [N, H * D] (the decay's pre-activation without its bias).  taps: float32 [C, n_taps], C = 2 G D + H V.
+// z: float32 rows of H * D, or of H with one decay per head (HEAD), row stride ld_z: the decay's pre-activation without its
+// bias (dt_bias has as many numbers as a row).  b_pre: the write strengths' pre-activations in float32 (row stride ld_z), or
+// null: the columns of proj at b_off.  taps: float32 [C, n_taps], C = 2 G D + H V.
 // Grid (N, G + H): CTA (t, u) with u < G prepares query/key head u of token t (convolution, silu, unit length, q . k);
 // with u >= G the values of head u - G (convolution, silu), that head's decays and its write strength -- so that a step of
 // a few single tokens still spreads over the GPU.
@@ -61,10 +65,10 @@ __device__ __forceinline__ float delta_conv(const A * __restrict__ proj, long lo
     return acc;
 }
 
-template <typename A>
+template <bool HEAD, typename A>
 __global__ void __launch_bounds__(kPrepThreads)
-delta_prep_kernel(const A * __restrict__ proj, long long ld, int col_off, int b_off,
-                  const float * __restrict__ z, const float * __restrict__ taps, int n_taps,
+delta_prep_kernel(const A * __restrict__ proj, long long ld, int col_off, int b_off, const float * __restrict__ b_pre,
+                  const float * __restrict__ z, long long ld_z, const float * __restrict__ taps, int n_taps,
                   const float * __restrict__ a_log, const float * __restrict__ dt_bias,
                   const float * __restrict__ state, long long state_stride, long long tail_off,
                   const int * __restrict__ seq_of_token, const int * __restrict__ cu_q,
@@ -125,11 +129,18 @@ delta_prep_kernel(const A * __restrict__ proj, long long ld, int col_off, int b_
         vv[t * HV + h * V + j] = silu_f32(delta_conv(proj, ld, col_off + c, (long long) t, first, tail, C, c, taps, n_taps));
     }
     const float rate = expf(a_log[h]);
-    for (int d = threadIdx.x; d < D; d += kPrepThreads) {
-        const size_t e = (size_t) h * D + d;
-        decay[t * (size_t) (H * D) + e] = expf(-rate * softplus_f32(z[t * (size_t) (H * D) + e] + dt_bias[e]));
+    if (HEAD) {
+        if (threadIdx.x == 0) decay[t * (size_t) H + h] = expf(-rate * softplus_f32(z[t * (size_t) ld_z + h] + dt_bias[h]));
+    } else {
+        for (int d = threadIdx.x; d < D; d += kPrepThreads) {
+            const size_t e = (size_t) h * D + d;
+            decay[t * (size_t) (H * D) + e] = expf(-rate * softplus_f32(z[t * (size_t) ld_z + e] + dt_bias[e]));
+        }
     }
-    if (threadIdx.x == 0) beta[t * H + h] = 1.0f / (1.0f + expf(-to_f32(proj[t * ld + b_off + h])));
+    if (threadIdx.x == 0) {
+        const float zb = b_pre != nullptr ? b_pre[t * (size_t) ld_z + h] : to_f32(proj[t * ld + b_off + h]);
+        beta[t * H + h] = 1.0f / (1.0f + expf(-zb));
+    }
 }
 
 // The same preparation for steps of many tokens.  Grid (ceil(N / T), G + H): a CTA takes T neighbouring rows of the step for
@@ -142,10 +153,10 @@ constexpr int kPrepTileWarps = 4;
 constexpr int kPrepTileFrom = 256;          // tokens in a step from which the tiled kernel runs (tiles of 8; of 16 from four times as many)
 constexpr int kPrepPerLane = kPrepMaxDim / 32;
 
-template <typename A>
+template <bool HEAD, typename A>
 __global__ void __launch_bounds__(kPrepTileWarps * 32)
-delta_prep_tile_kernel(const A * __restrict__ proj, long long ld, int col_off, int b_off,
-                       const float * __restrict__ z, const float * __restrict__ taps, int n_taps,
+delta_prep_tile_kernel(const A * __restrict__ proj, long long ld, int col_off, int b_off, const float * __restrict__ b_pre,
+                       const float * __restrict__ z, long long ld_z, const float * __restrict__ taps, int n_taps,
                        const float * __restrict__ a_log, const float * __restrict__ dt_bias,
                        const float * __restrict__ state, long long state_stride, long long tail_off,
                        const int * __restrict__ seq_of_token, const int * __restrict__ cu_q,
@@ -246,13 +257,20 @@ delta_prep_tile_kernel(const A * __restrict__ proj, long long ld, int col_off, i
         } else {
             const int h = u - G;
             const float rate = expf(a_log[h]);
-            for (int d = lane; d < D; d += 32) {
-                const size_t e = (size_t) h * D + d;
-                decay[t * (size_t) HD + e] = expf(-rate * softplus_f32(z[t * (size_t) HD + e] + dt_bias[e]));
+            if (HEAD) {
+                if (lane == 0) decay[t * (size_t) H + h] = expf(-rate * softplus_f32(z[t * (size_t) ld_z + h] + dt_bias[h]));
+            } else {
+                for (int d = lane; d < D; d += 32) {
+                    const size_t e = (size_t) h * D + d;
+                    decay[t * (size_t) HD + e] = expf(-rate * softplus_f32(z[t * (size_t) ld_z + e] + dt_bias[e]));
+                }
             }
             for (int j = lane; j < V; j += 32)
                 vv[t * HV + h * V + j] = silu_f32(conv(ti, before, tail, j, 2 * GD + h * V + j));
-            if (lane == 0) beta[t * H + h] = 1.0f / (1.0f + expf(-to_f32(proj[t * ld + b_off + h])));
+            if (lane == 0) {
+                const float zb = b_pre != nullptr ? b_pre[t * (size_t) ld_z + h] : to_f32(proj[t * ld + b_off + h]);
+                beta[t * H + h] = 1.0f / (1.0f + expf(-zb));
+            }
         }
     }
 }
@@ -276,7 +294,8 @@ template <int N> __device__ __forceinline__ void dr_wait() { asm volatile("cp.as
 // neighbouring entries, d = 4 * lane + 32 * (i / 4) + i % 4, so that the state and the rows of q, k and the decays move
 // 16 bytes at a time (E a multiple of 4); else entry d = lane + kLanes * i, word by word.  The tokens of a sequence pass
 // through two stages of shared memory, `chunk` tokens each: while one is worked through, cp.async fills the other.
-template <int E, bool VEC, typename A>
+// HEAD: one decay per (token, head), decay [N, H]; it sits beside the write strength and q . k of its token.
+template <int E, bool VEC, bool HEAD, typename A>
 __global__ void __launch_bounds__(kCols * kLanes)
 delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, const float * __restrict__ vv,
                   const float * __restrict__ beta, const float * __restrict__ decay, const float * __restrict__ qk,
@@ -288,7 +307,7 @@ delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, 
     pdl_launch_dependents();
     extern __shared__ __align__(16) float sm[];
     const int Dp = (D + 3) & ~3;                             // rows start on 16-byte boundaries
-    const int stage_floats = chunk * (3 * Dp + kCols + 4);   // q | k | decay | v | beta, q . k (padded to 4 per token)
+    const int stage_floats = chunk * ((HEAD ? 2 : 3) * Dp + kCols + 4);      // q | k | decay (not HEAD) | v | beta, q . k, decay (HEAD), -
     const int cb = blockIdx.x, h = blockIdx.y, s = blockIdx.z;
     const int g = h / (H / G);
     const int col = threadIdx.x / kLanes, lane = threadIdx.x % kLanes;
@@ -296,6 +315,7 @@ delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, 
     const int t0 = cu_q[s], t1 = cu_q[s + 1];
     const int slot = state_slots[s];
     const int HV = H * V, GD = G * D, HD = H * D;
+    constexpr int kPer = HEAD ? 4 : 2;         // numbers per token behind the values
     if (slot < 0) {                            // a padding sequence: zeros out, nothing kept
         for (int t = t0; t < t1; t++)
             if (lane == 0 && j < V) out[(size_t) t * HV + h * V + j] = 0.0f;
@@ -308,7 +328,7 @@ delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, 
         float * s_q = sm + (size_t) stage * stage_floats;
         float * s_k = s_q + chunk * Dp;
         float * s_g = s_k + chunk * Dp;
-        float * s_v = s_g + chunk * Dp;
+        float * s_v = s_g + (HEAD ? 0 : chunk * Dp);
         float * s_b = s_v + chunk * kCols;
         if (VEC) {
             const int per = D >> 2;
@@ -317,7 +337,7 @@ delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, 
                 const size_t t = c0 + tt;
                 dr_cp16(s_q + tt * Dp + d, qn + t * GD + g * D + d);
                 dr_cp16(s_k + tt * Dp + d, kn + t * GD + g * D + d);
-                dr_cp16(s_g + tt * Dp + d, decay + t * HD + h * D + d);
+                if (!HEAD) dr_cp16(s_g + tt * Dp + d, decay + t * HD + h * D + d);
             }
         } else {
             for (int e = threadIdx.x; e < nt * D; e += blockDim.x) {
@@ -325,7 +345,7 @@ delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, 
                 const size_t t = c0 + tt;
                 dr_cp4(s_q + tt * Dp + d, qn + t * GD + g * D + d, true);
                 dr_cp4(s_k + tt * Dp + d, kn + t * GD + g * D + d, true);
-                dr_cp4(s_g + tt * Dp + d, decay + t * HD + h * D + d, true);
+                if (!HEAD) dr_cp4(s_g + tt * Dp + d, decay + t * HD + h * D + d, true);
             }
         }
         for (int e = threadIdx.x; e < nt * kCols; e += blockDim.x) {
@@ -334,8 +354,9 @@ delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, 
             dr_cp4(s_v + e, vv + (size_t) (c0 + tt) * HV + h * V + (jj < V ? jj : 0), jj < V);
         }
         for (int e = threadIdx.x; e < nt; e += blockDim.x) {
-            dr_cp4(s_b + 2 * e, beta + (size_t) (c0 + e) * H + h, true);
-            dr_cp4(s_b + 2 * e + 1, qk + (size_t) (c0 + e) * G + g, true);
+            dr_cp4(s_b + kPer * e, beta + (size_t) (c0 + e) * H + h, true);
+            dr_cp4(s_b + kPer * e + 1, qk + (size_t) (c0 + e) * G + g, true);
+            if (HEAD) dr_cp4(s_b + kPer * e + 2, decay + (size_t) (c0 + e) * H + h, true);
         }
     };
     if (t0 < t1) fill(t0, 0);
@@ -394,7 +415,7 @@ delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, 
         const float * s_q = sm + (size_t) stage * stage_floats;
         const float * s_k = s_q + chunk * Dp;
         const float * s_g = s_k + chunk * Dp;
-        const float * s_v = s_g + chunk * Dp;
+        const float * s_v = s_g + (HEAD ? 0 : chunk * Dp);
         const float * s_b = s_v + chunk * kCols;
         for (int tt = 0; tt < nt; tt++) {
             const float * kq = s_k + tt * Dp;
@@ -408,12 +429,12 @@ delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, 
                     const int d = 4 * lane + 4 * kLanes * (i >> 2);
                     float4 g4 = make_float4(1.0f, 1.0f, 1.0f, 1.0f), k4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f), q4 = k4;
                     if (d < D) {
-                        g4 = *reinterpret_cast<const float4 *>(gg + d);
+                        if (!HEAD) g4 = *reinterpret_cast<const float4 *>(gg + d);
                         k4 = *reinterpret_cast<const float4 *>(kq + d);
                         q4 = *reinterpret_cast<const float4 *>(qq + d);
                     }
                     kk[i] = k4.x; kk[i + 1] = k4.y; kk[i + 2] = k4.z; kk[i + 3] = k4.w;
-                    S[i] *= g4.x; S[i + 1] *= g4.y; S[i + 2] *= g4.z; S[i + 3] *= g4.w;
+                    if (!HEAD) { S[i] *= g4.x; S[i + 1] *= g4.y; S[i + 2] *= g4.z; S[i + 3] *= g4.w; }
                     a0 = fmaf(k4.x, S[i], a0);     b0 = fmaf(q4.x, S[i], b0);
                     a1 = fmaf(k4.y, S[i + 1], a1); b1 = fmaf(q4.y, S[i + 1], b1);
                     a0 = fmaf(k4.z, S[i + 2], a0); b0 = fmaf(q4.z, S[i + 2], b0);
@@ -426,13 +447,13 @@ delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, 
                     kk[i] = kk[i + 1] = 0.0f;
                     if (d < D) {
                         kk[i] = kq[d];
-                        S[i] *= gg[d];
+                        if (!HEAD) S[i] *= gg[d];
                         a0 = fmaf(kk[i], S[i], a0);
                         b0 = fmaf(qq[d], S[i], b0);
                     }
                     if (d + kLanes < D) {
                         kk[i + 1] = kq[d + kLanes];
-                        S[i + 1] *= gg[d + kLanes];
+                        if (!HEAD) S[i + 1] *= gg[d + kLanes];
                         a1 = fmaf(kk[i + 1], S[i + 1], a1);
                         b1 = fmaf(qq[d + kLanes], S[i + 1], b1);
                     }
@@ -444,10 +465,12 @@ delta_scan_kernel(const float * __restrict__ qn, const float * __restrict__ kn, 
                 a += __shfl_xor_sync(0xffffffffu, a, o);
                 b += __shfl_xor_sync(0xffffffffu, b, o);
             }
-            const float u = s_b[2 * tt] * (s_v[tt * kCols + col] - a);
+            const float gd = HEAD ? s_b[kPer * tt + 2] : 1.0f;
+            if (HEAD) { a *= gd; b *= gd; }
+            const float u = s_b[kPer * tt] * (s_v[tt * kCols + col] - a);
 #pragma unroll
-            for (int i = 0; i < E; i++) S[i] = fmaf(kk[i], u, S[i]);        // (entries beyond D stay zero: their key is zero)
-            if (lane == 0 && j < V) out[(size_t) (c0 + tt) * HV + h * V + j] = fmaf(s_b[2 * tt + 1], u, b);
+            for (int i = 0; i < E; i++) S[i] = fmaf(kk[i], u, HEAD ? gd * S[i] : S[i]);     // (entries beyond D stay zero: their key is zero)
+            if (lane == 0 && j < V) out[(size_t) (c0 + tt) * HV + h * V + j] = fmaf(s_b[kPer * tt + 1], u, b);
         }
         __syncthreads();                       // everyone is done with this stage before it is filled again
     }
@@ -477,15 +500,12 @@ IIAN_API long long iian_delta_state_floats(int H, int G, int D, int V, int n_tap
     return (long long) H * V * D + (long long) (n_taps - 1) * (2LL * G * D + (long long) H * V);
 }
 
-IIAN_API int iian_delta_prep(const void * proj, long long ld, int col_off, int b_off, int act_dtype, const float * z,
-                             const float * taps, int n_taps, const float * a_log, const float * dt_bias, const float * state,
-                             long long state_stride, const int * seq_of_token, const int * cu_q, const int * state_slots,
-                             float * qn, float * kn, float * vv, float * beta, float * decay, float * qk, int N, int H, int G,
-                             int D, int V, cudaStream_t stream) {
-    if (N <= 0) return IIAN_OK;
-    if (H <= 0 || G <= 0 || H % G || D <= 0 || V <= 0 || n_taps < 1 || n_taps > kMaxTaps) return IIAN_ERR_SHAPE;
-    if (D > kPrepMaxDim) return IIAN_ERR_LIMIT;
-    if (G + H > 65535) return IIAN_ERR_LIMIT;
+template <bool HEAD, typename A>
+static int launch_prep(const A * proj, long long ld, int col_off, int b_off, const float * b_pre, const float * z, long long ld_z,
+                       const float * taps, int n_taps, const float * a_log, const float * dt_bias, const float * state,
+                       long long state_stride, const int * seq_of_token, const int * cu_q, const int * state_slots, float * qn,
+                       float * kn, float * vv, float * beta, float * decay, float * qk, int N, int H, int G, int D, int V,
+                       cudaStream_t stream) {
     const long long tail_off = (long long) H * V * D;
     const float q_scale = 1.0f / sqrtf((float) D);
     // many tokens: tiles of T rows through shared memory; few: a CTA per token and unit, so that they spread over the GPU
@@ -498,33 +518,37 @@ IIAN_API int iian_delta_prep(const void * proj, long long ld, int col_off, int b
     }
     if (T >= 4) {
         const dim3 tgrid((N + T - 1) / T, G + H);
-        if (act_dtype == IIAN_F32) {
-            if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prep_tile_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
-            return iian_launch(delta_prep_tile_kernel<float>, tgrid, dim3(kPrepTileWarps * 32), smem, stream, (const float *) proj, ld,
-                               col_off, b_off, z, taps, n_taps, a_log, dt_bias, state, state_stride, tail_off, seq_of_token, cu_q,
-                               state_slots, qn, kn, vv, beta, decay, qk, N, T, H, G, D, V, q_scale);
-        }
-        if (act_dtype == IIAN_BF16) {
-            if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prep_tile_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
-            return iian_launch(delta_prep_tile_kernel<__nv_bfloat16>, tgrid, dim3(kPrepTileWarps * 32), smem, stream,
-                               (const __nv_bfloat16 *) proj, ld, col_off, b_off, z, taps, n_taps, a_log, dt_bias, state, state_stride,
-                               tail_off, seq_of_token, cu_q, state_slots, qn, kn, vv, beta, decay, qk, N, T, H, G, D, V, q_scale);
-        }
-        return IIAN_ERR_DTYPE;
+        if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prep_tile_kernel<HEAD, A>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
+        return iian_launch(delta_prep_tile_kernel<HEAD, A>, tgrid, dim3(kPrepTileWarps * 32), smem, stream, proj, ld, col_off, b_off, b_pre,
+                           z, ld_z, taps, n_taps, a_log, dt_bias, state, state_stride, tail_off, seq_of_token, cu_q, state_slots, qn, kn,
+                           vv, beta, decay, qk, N, T, H, G, D, V, q_scale);
     }
-    const dim3 grid(N, G + H);
-    if (act_dtype == IIAN_F32)
-        return iian_launch(delta_prep_kernel<float>, grid, dim3(kPrepThreads), 0, stream, (const float *) proj, ld, col_off, b_off, z,
-                           taps, n_taps, a_log, dt_bias, state, state_stride, tail_off, seq_of_token, cu_q, state_slots, qn, kn,
-                           vv, beta, decay, qk, H, G, D, V, q_scale);
-    if (act_dtype == IIAN_BF16)
-        return iian_launch(delta_prep_kernel<__nv_bfloat16>, grid, dim3(kPrepThreads), 0, stream, (const __nv_bfloat16 *) proj, ld,
-                           col_off, b_off, z, taps, n_taps, a_log, dt_bias, state, state_stride, tail_off, seq_of_token, cu_q,
-                           state_slots, qn, kn, vv, beta, decay, qk, H, G, D, V, q_scale);
+    return iian_launch(delta_prep_kernel<HEAD, A>, dim3(N, G + H), dim3(kPrepThreads), 0, stream, proj, ld, col_off, b_off, b_pre, z, ld_z,
+                       taps, n_taps, a_log, dt_bias, state, state_stride, tail_off, seq_of_token, cu_q, state_slots, qn, kn, vv, beta,
+                       decay, qk, H, G, D, V, q_scale);
+}
+
+// per_head: one decay per head (z, dt_bias and decay hold H numbers per token) instead of one per key channel (H * D).
+// b_pre: float32 pre-activations of the write strengths (row stride ld_z), or null: the columns of proj at b_off.
+IIAN_API int iian_delta_prep(const void * proj, long long ld, int col_off, int b_off, int act_dtype, const float * b_pre, const float * z,
+                             long long ld_z, int per_head, const float * taps, int n_taps, const float * a_log, const float * dt_bias,
+                             const float * state, long long state_stride, const int * seq_of_token, const int * cu_q,
+                             const int * state_slots, float * qn, float * kn, float * vv, float * beta, float * decay, float * qk,
+                             int N, int H, int G, int D, int V, cudaStream_t stream) {
+    if (N <= 0) return IIAN_OK;
+    if (H <= 0 || G <= 0 || H % G || D <= 0 || V <= 0 || n_taps < 1 || n_taps > kMaxTaps) return IIAN_ERR_SHAPE;
+    if (D > kPrepMaxDim) return IIAN_ERR_LIMIT;
+    if (G + H > 65535) return IIAN_ERR_LIMIT;
+#define IIAN_PREP(HEAD, A) return launch_prep<HEAD, A>((const A *) proj, ld, col_off, b_off, b_pre, z, ld_z, taps, n_taps, a_log, dt_bias, \
+                                                       state, state_stride, seq_of_token, cu_q, state_slots, qn, kn, vv, beta, decay, qk, \
+                                                       N, H, G, D, V, stream)
+    if (act_dtype == IIAN_F32) { if (per_head) IIAN_PREP(true, float); IIAN_PREP(false, float); }
+    if (act_dtype == IIAN_BF16) { if (per_head) IIAN_PREP(true, __nv_bfloat16); IIAN_PREP(false, __nv_bfloat16); }
+#undef IIAN_PREP
     return IIAN_ERR_DTYPE;
 }
 
-template <int E, typename A>
+template <int E, bool HEAD, typename A>
 static int launch_scan(const float * qn, const float * kn, const float * vv, const float * beta, const float * decay,
                        const float * qk, float * state, long long state_stride, const A * proj, long long ld, int col_off,
                        int n_taps, const int * cu_q, const int * state_slots, float * out, int S, int H, int G, int D, int V,
@@ -532,20 +556,20 @@ static int launch_scan(const float * qn, const float * kn, const float * vv, con
     const int Dp = (D + 3) & ~3;
     int chunk = D <= 256 ? 16 : 8;             // tokens per stage of shared memory
     if (max_q_len > 0 && max_q_len < chunk) chunk = max_q_len;         // single tokens: small stages, more CTAs per SM
-    const size_t smem = (size_t) 2 * chunk * (3 * Dp + kCols + 4) * sizeof(float);
+    const size_t smem = (size_t) 2 * chunk * ((HEAD ? 2 : 3) * Dp + kCols + 4) * sizeof(float);
     if (smem > 200 * 1024) return IIAN_ERR_LIMIT;
     const dim3 grid((V + kCols - 1) / kCols, H, S);
     if constexpr (E % 4 == 0) if (vec) {
-        if (smem > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<E, true, A>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
-        return iian_launch(delta_scan_kernel<E, true, A>, grid, dim3(kCols * kLanes), smem, stream, qn, kn, vv, beta, decay, qk, state,
+        if (smem > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<E, true, HEAD, A>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
+        return iian_launch(delta_scan_kernel<E, true, HEAD, A>, grid, dim3(kCols * kLanes), smem, stream, qn, kn, vv, beta, decay, qk, state,
                            state_stride, (long long) H * V * D, proj, ld, col_off, n_taps, cu_q, state_slots, out, H, G, D, V, chunk);
     }
-    if (smem > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<E, false, A>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
-    return iian_launch(delta_scan_kernel<E, false, A>, grid, dim3(kCols * kLanes), smem, stream, qn, kn, vv, beta, decay, qk, state,
+    if (smem > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<E, false, HEAD, A>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
+    return iian_launch(delta_scan_kernel<E, false, HEAD, A>, grid, dim3(kCols * kLanes), smem, stream, qn, kn, vv, beta, decay, qk, state,
                        state_stride, (long long) H * V * D, proj, ld, col_off, n_taps, cu_q, state_slots, out, H, G, D, V, chunk);
 }
 
-template <typename A>
+template <bool HEAD, typename A>
 static int scan_by_depth(const float * qn, const float * kn, const float * vv, const float * beta, const float * decay,
                          const float * qk, float * state, long long state_stride, const A * proj, long long ld, int col_off,
                          int n_taps, const int * cu_q, const int * state_slots, float * out, int S, int H, int G, int D, int V,
@@ -553,7 +577,7 @@ static int scan_by_depth(const float * qn, const float * kn, const float * vv, c
     const int e = (D + kLanes - 1) / kLanes;
     const bool vec = D % 4 == 0 && state_stride % 4 == 0 &&
                      (((uintptr_t) qn | (uintptr_t) kn | (uintptr_t) decay | (uintptr_t) state) & 15) == 0;
-#define IIAN_SCAN(E) return launch_scan<E, A>(qn, kn, vv, beta, decay, qk, state, state_stride, proj, ld, col_off, n_taps, cu_q, \
+#define IIAN_SCAN(E) return launch_scan<E, HEAD, A>(qn, kn, vv, beta, decay, qk, state, state_stride, proj, ld, col_off, n_taps, cu_q, \
                                               state_slots, out, S, H, G, D, V, max_q_len, vec, stream)
     if (e <= 2 && !vec) IIAN_SCAN(2);
     if (e <= 4) IIAN_SCAN(4);
@@ -565,19 +589,19 @@ static int scan_by_depth(const float * qn, const float * kn, const float * vv, c
     return IIAN_ERR_LIMIT;
 }
 
-// out: float32 [N, H * V].  S sequences (grid z); a sequence with state slot -1 is padding.  max_q_len: the most tokens a
+// out: float32 [N, H * V].  per_head: decay is [N, H] instead of [N, H * D].  S sequences (grid z); a sequence with state slot -1 is padding.  max_q_len: the most tokens a
 // sequence has in this step (0: unknown); it sizes the stages of shared memory.
 IIAN_API int iian_delta_scan(const float * qn, const float * kn, const float * vv, const float * beta, const float * decay,
                              const float * qk, float * state, long long state_stride, const void * proj, long long ld,
                              int col_off, int act_dtype, int n_taps, const int * cu_q, const int * state_slots, float * out,
-                             int S, int H, int G, int D, int V, int max_q_len, cudaStream_t stream) {
+                             int S, int H, int G, int D, int V, int max_q_len, int per_head,
+                            cudaStream_t stream) {
     if (S <= 0) return IIAN_OK;
     if (H <= 0 || G <= 0 || H % G || D <= 0 || V <= 0 || n_taps < 1 || n_taps > kMaxTaps || S > 65535 || H > 65535) return IIAN_ERR_SHAPE;
-    if (act_dtype == IIAN_F32)
-        return scan_by_depth<float>(qn, kn, vv, beta, decay, qk, state, state_stride, (const float *) proj, ld, col_off, n_taps,
-                                    cu_q, state_slots, out, S, H, G, D, V, max_q_len, stream);
-    if (act_dtype == IIAN_BF16)
-        return scan_by_depth<__nv_bfloat16>(qn, kn, vv, beta, decay, qk, state, state_stride, (const __nv_bfloat16 *) proj, ld,
-                                            col_off, n_taps, cu_q, state_slots, out, S, H, G, D, V, max_q_len, stream);
+#define IIAN_SCAN_AS(HEAD, A) return scan_by_depth<HEAD, A>(qn, kn, vv, beta, decay, qk, state, state_stride, (const A *) proj, ld, col_off, \
+                                                            n_taps, cu_q, state_slots, out, S, H, G, D, V, max_q_len, stream)
+    if (act_dtype == IIAN_F32) { if (per_head) IIAN_SCAN_AS(true, float); IIAN_SCAN_AS(false, float); }
+    if (act_dtype == IIAN_BF16) { if (per_head) IIAN_SCAN_AS(true, __nv_bfloat16); IIAN_SCAN_AS(false, __nv_bfloat16); }
+#undef IIAN_SCAN_AS
     return IIAN_ERR_DTYPE;
 }

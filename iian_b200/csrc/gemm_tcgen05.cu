@@ -30,7 +30,7 @@ constexpr int TC_BK = 64;                 // 64 bf16 = 128 bytes = one swizzle a
 constexpr int TC_THREADS = 192;           // warp 0: TMA, warp 1: MMA + TMEM, warps 2..5: epilogue
 constexpr unsigned kSpinLimit = 2u * 1000u * 1000u;
 
-enum { EPI_STORE = 0, EPI_SWIGLU8 = 1, EPI_RESNORM = 2 };
+enum { EPI_STORE = 0, EPI_SWIGLU8 = 1, EPI_RESNORM = 2, EPI_RELU2 = 3 };      // EPI_RELU2 (grouped form): max(z, 0)^2
 
 struct TcStatus { int code; int where; };
 
@@ -133,7 +133,14 @@ __device__ __forceinline__ void epilogue_store32(unsigned * r, OutT * __restrict
 #pragma unroll
         for (int i = 0; i < 32; i++) r[i] = __float_as_uint(__uint_as_float(r[i]) * rs);
     }
-    if (EPI == EPI_STORE) {
+    if (EPI == EPI_RELU2) {
+#pragma unroll
+        for (int i = 0; i < 32; i++) {
+            const float z = fmaxf(__uint_as_float(r[i]), 0.0f);
+            r[i] = __float_as_uint(z * z);
+        }
+    }
+    if (EPI == EPI_STORE || EPI == EPI_RELU2) {
         OutT * dst = out + (size_t) row * ldo + col0;
         if (col0 + 32 <= N && (((uintptr_t) dst) & 15) == 0) {
             if (sizeof(OutT) == 2) {
@@ -680,7 +687,7 @@ static int tc_entry(const void * x, const void * w, void * out, int out_dtype, i
 }
 
 // The grouped product: x [T, K] bf16 with its rows sorted by group, w [groups * N, K] bf16 (group e's matrix in rows
-// e * N ..), out [T, N] or, with epilogue 1, [T, N / 2]; tiles = {row tiles, then (group, first row) per row tile of 128
+// e * N ..), out [T, N] or, with epilogue 1, [T, N / 2] (epilogue 3: max(z, 0)^2 of every entry); tiles = {row tiles, then (group, first row) per row tile of 128
 // rows}, offsets [groups + 1], both on the device; max_tiles bounds the row tiles (it sizes the grid).  bn: 128 or 256.
 IIAN_API int iian_gemm_tcgen05_grouped(const void * x, const void * w, void * out, int out_dtype, int T, int N, int groups, int K,
                                        int epilogue, int bn, int * status, const int * tiles, const int * offsets, int max_tiles,
@@ -688,7 +695,7 @@ IIAN_API int iian_gemm_tcgen05_grouped(const void * x, const void * w, void * ou
     if (T <= 0 || N <= 0 || groups <= 0 || max_tiles <= 0) return IIAN_OK;
     if (K <= 0 || K % 8 != 0 || tiles == nullptr || offsets == nullptr || status == nullptr) return IIAN_ERR_SHAPE;
     if (((uintptr_t) x & 15) || ((uintptr_t) w & 15)) return IIAN_ERR_ALIGN;
-    if (epilogue != EPI_STORE && epilogue != EPI_SWIGLU8) return IIAN_ERR_SHAPE;
+    if (epilogue != EPI_STORE && epilogue != EPI_SWIGLU8 && epilogue != EPI_RELU2) return IIAN_ERR_SHAPE;
     if (epilogue == EPI_SWIGLU8 && N % 16 != 0) return IIAN_ERR_SHAPE;
     if (bn != 128 && bn != 256) return IIAN_ERR_SHAPE;
     if (out_dtype != IIAN_BF16) return IIAN_ERR_DTYPE;
@@ -701,6 +708,9 @@ IIAN_API int iian_gemm_tcgen05_grouped(const void * x, const void * w, void * ou
     TcStatus * st = (TcStatus *) status;
     const int ldo = epilogue == EPI_SWIGLU8 ? N / 2 : N;
     const TcExtra ex = {nullptr, 0, 0.0f, 0.0f, nullptr, nullptr, nullptr, tiles, offsets, N};
+    if (epilogue == EPI_RELU2)
+        return bn == 256 ? launch_tc<256, 4, EPI_RELU2, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream, max_tiles)
+                         : launch_tc<128, 6, EPI_RELU2, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream, max_tiles);
     if (bn == 256)
         return epilogue == EPI_STORE ? launch_tc<256, 4, EPI_STORE, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream, max_tiles)
                                      : launch_tc<256, 4, EPI_SWIGLU8, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream, max_tiles);

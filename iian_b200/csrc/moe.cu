@@ -60,6 +60,46 @@ __global__ void moe_route_kernel(const float * __restrict__ logits, long long ld
     }
 }
 
+// Scores s = softmax(z) over all E outputs; a token takes the `top` outputs with the largest s + correction (ties: lowest
+// index); each weighs scale * s (without the correction, not renormalised).  One warp per token.
+__global__ void moe_route_corrected_kernel(const float * __restrict__ logits, long long ld, const float * __restrict__ correction,
+                                           int E, int top, int * __restrict__ ids, float * __restrict__ wts, int N, float scale) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const long long t = (long long) blockIdx.x * (blockDim.x >> 5) + warp;
+    if (t >= N) return;
+    const float * z = logits + t * ld;
+    float mx = -INFINITY;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+    mx = warp_max(mx);
+    float sum = 0.0f;
+    for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
+    sum = warp_sum(sum);
+    unsigned long long taken = 0;              // this lane's outputs already chosen, by slot e / 32
+    for (int k = 0; k < top; k++) {
+        float best = -INFINITY, best_s = 0.0f;
+        int best_e = 0x7fffffff;
+        for (int e = lane, i = 0; e < E; e += 32, i++) {
+            if ((taken >> i) & 1ull) continue;
+            const float s = expf(z[e] - mx) / sum;
+            const float v = correction != nullptr ? s + correction[e] : s;
+            if (v > best || best_e == 0x7fffffff) { best = v; best_s = s; best_e = e; }        // (a lane's e rise: ties keep the lower)
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, best, o), os = __shfl_xor_sync(0xffffffffu, best_s, o);
+            const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
+            if (oe != 0x7fffffff && (best_e == 0x7fffffff || ov > best || (ov == best && oe < best_e))) { best = ov; best_s = os; best_e = oe; }
+        }
+        if (best_e != 0x7fffffff && (best_e & 31) == lane) taken |= 1ull << (best_e >> 5);
+        if (lane == 0) {
+            ids[t * top + k] = best_e == 0x7fffffff ? 0 : best_e;
+            wts[t * top + k] = best_e == 0x7fffffff ? 0.0f : scale * best_s;
+        }
+    }
+}
+
 // Routing without a router: row `tokens[t]` of a table [V, top] names the token's experts (the entries of a row differ);
 // each weighs `weight`.  rows (optional): the token of output row r is tokens[rows[r]].
 __global__ void moe_table_route_kernel(const int * __restrict__ tokens, const int * __restrict__ rows, const int * __restrict__ table,
@@ -77,7 +117,8 @@ __global__ void moe_table_route_kernel(const int * __restrict__ tokens, const in
     wts[i] = weight;
 }
 
-// One block.  offsets: [E + 1] first sorted row of each expert; pos: [M] sorted row of each (token, choice);
+// One block.  A choice ids[i] >= E has no expert behind it (an output that passes its input on): it gets no row, pos[i] = -1.
+// offsets: [E + 1] first sorted row of each expert; pos: [M] sorted row of each (token, choice);
 // tiles: [2 * max_tiles + 1]: n_tiles, then (expert, first row) per row tile of tile_rows rows.
 __global__ void moe_plan_kernel(const int * __restrict__ ids, int M, int E, int * __restrict__ offsets, int * __restrict__ pos,
                                 int * __restrict__ tiles, int max_tiles, int tile_rows) {
@@ -88,7 +129,8 @@ __global__ void moe_plan_kernel(const int * __restrict__ ids, int M, int E, int 
     int * cursor = sm + E;
     for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
     __syncthreads();
-    for (int i = threadIdx.x; i < M; i += blockDim.x) atomicAdd(&counts[ids[i]], 1);
+    for (int i = threadIdx.x; i < M; i += blockDim.x)
+        if ((unsigned) ids[i] < (unsigned) E) atomicAdd(&counts[ids[i]], 1);
     __syncthreads();
     if (threadIdx.x == 0) {
         int run = 0, nt = 0;
@@ -107,7 +149,7 @@ __global__ void moe_plan_kernel(const int * __restrict__ ids, int M, int E, int 
     }
     __syncthreads();
     // the order of an expert's rows among themselves is left to the atomics: a row's arithmetic does not depend on it
-    for (int i = threadIdx.x; i < M; i += blockDim.x) pos[i] = atomicAdd(&cursor[ids[i]], 1);
+    for (int i = threadIdx.x; i < M; i += blockDim.x) pos[i] = (unsigned) ids[i] < (unsigned) E ? atomicAdd(&cursor[ids[i]], 1) : -1;
 }
 
 // xs[pos[t * top + k], :] = A(w[t, k] * h[t, :]);  rows[pos] = t * top + k
@@ -118,6 +160,7 @@ __global__ void moe_scatter_kernel(const A * __restrict__ h, const int * __restr
     pdl_launch_dependents();
     const size_t i = blockIdx.x;              // (token, choice)
     const size_t t = i / top;
+    if (pos[i] < 0) return;                   // no expert behind this choice
     const float w = wts != nullptr ? wts[i] : 1.0f;
     const A * src = h + t * W;
     A * dst = xs + (size_t) pos[i] * W;
@@ -142,6 +185,52 @@ __global__ void moe_combine_kernel(const A * __restrict__ ys, const int * __rest
     }
 }
 
+// The same for outputs some of which pass their input on (pos < 0: the row h[t] itself takes the place of an expert's output)
+// and an addend with a factor per token: out[t, :] = sum_k wts[t, k] * (pos >= 0 ? ys[pos] : h[t]) [+ sigmoid(add_gate[t]) *
+// add[t, :]], k ascending, float32.  A thread takes V neighbouring columns (V = 1 or 8 bf16 / 4 f32: 16 bytes).
+template <typename A, int V>
+__global__ void moe_combine_mixed_kernel(const A * __restrict__ ys, const int * __restrict__ pos, const float * __restrict__ wts,
+                                         const A * __restrict__ h, A * out, int W, int top, const A * add,
+                                         const float * __restrict__ add_gate, long long ld_gate) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t t = blockIdx.x;
+    const float ag = add_gate != nullptr ? 1.0f / (1.0f + expf(-add_gate[t * ld_gate])) : 1.0f;
+    for (int c = V * (blockIdx.y * blockDim.x + threadIdx.x); c < W; c += V * blockDim.x * gridDim.y) {
+        float acc[V];
+#pragma unroll
+        for (int i = 0; i < V; i++) acc[i] = 0.0f;
+        auto take = [&](const A * src, float w) {
+            if constexpr (V == 8) {
+                float f[8];
+                unpack8(*reinterpret_cast<const uint4 *>(src), f);
+#pragma unroll
+                for (int i = 0; i < 8; i++) acc[i] = fmaf(w, f[i], acc[i]);
+            } else if constexpr (V == 4) {
+                const float4 f = *reinterpret_cast<const float4 *>(src);
+                acc[0] = fmaf(w, f.x, acc[0]); acc[1] = fmaf(w, f.y, acc[1]); acc[2] = fmaf(w, f.z, acc[2]); acc[3] = fmaf(w, f.w, acc[3]);
+            } else {
+                acc[0] = fmaf(w, to_f32(*src), acc[0]);
+            }
+        };
+        for (int k = 0; k < top; k++) {
+            const int p = pos[t * top + k];
+            take(p >= 0 ? ys + (size_t) p * W + c : h + t * W + c, wts[t * top + k]);
+        }
+        if (add != nullptr) take(add + t * W + c, ag);            // may be `out` itself: read before it is written
+        if constexpr (V == 8) {
+            __nv_bfloat162 r[4];
+#pragma unroll
+            for (int i = 0; i < 4; i++) r[i] = __floats2bfloat162_rn(acc[2 * i], acc[2 * i + 1]);
+            *reinterpret_cast<uint4 *>(out + t * W + c) = *reinterpret_cast<uint4 *>(r);
+        } else if constexpr (V == 4) {
+            *reinterpret_cast<float4 *>(out + t * W + c) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        } else {
+            out[t * W + c] = from_f32<A>(acc[0]);
+        }
+    }
+}
+
 // act 0: silu(g) * u; 1: gelu_tanh(g) * u; 2: with g' = min(g, limit), u' = clamp(u, -limit, limit):
 // g' sigmoid(1.702 g') (u' + 1)
 __device__ __forceinline__ float moe_gated(float g, float u, int act, float limit) {
@@ -157,7 +246,7 @@ __device__ __forceinline__ float moe_gated(float g, float u, int act, float limi
 
 // Rows [r0, r0 + rows) of x (sorted by expert) times expert e's weight block w[e] ([n_out, K], row-major):
 // out[r, m] = sum_k x[r, k] * w[e][m, k];  with GATED, w2[e] is a second block of the same shape and
-// out[r, m] = act(x . w[e][m]) * (x . w2[e][m]); with GATED and w2 == w, an expert's block holds both, 2 n_out rows in
+// out[r, m] = act(x . w[e][m]) * (x . w2[e][m]); without, act 3 squares the positive part; with GATED and w2 == w, an expert's block holds both, 2 n_out rows in
 // groups of 16: 8 rows of the first, then the 8 rows of the second for the same features.
 template <typename A, typename WT, bool GATED>
 __global__ void __launch_bounds__(256) moe_grouped_gemm_kernel(const A * __restrict__ x, const WT * __restrict__ w,
@@ -229,6 +318,7 @@ __global__ void __launch_bounds__(256) moe_grouped_gemm_kernel(const A * __restr
             float v = acc[i][j];
             // the gate and up products are rounded to the activation type first, as separate products would leave them
             if (GATED) v = moe_gated(to_f32(from_f32<A>(v)), to_f32(from_f32<A>(acc2[i][j])), act, limit);
+            else if (act == 3) { v = fmaxf(v, 0.0f); v *= v; }
             out[(size_t) r * n_out + m] = from_f32<A>(v);
         }
     }
@@ -257,6 +347,16 @@ IIAN_API int iian_moe_route_softmax(const float * logits, long long ld, const fl
     const int warps = 4;
     return iian_launch(moe_route_kernel, dim3((N + warps - 1) / warps), dim3(warps * 32), 0, stream, logits, ld, E, top, ids, wts, N,
                        bias, 1);
+}
+
+// Softmax over all E outputs, choice by score + correction (float32 [E] or null), weights scale * score.
+IIAN_API int iian_moe_route_corrected(const float * logits, long long ld, const float * correction, int E, int top, int * ids,
+                                      float * wts, float scale, int N, cudaStream_t stream) {
+    if (N <= 0) return IIAN_OK;
+    if (E <= 0 || top <= 0 || top > E || E > 2048) return IIAN_ERR_SHAPE;
+    const int warps = 4;
+    return iian_launch(moe_route_corrected_kernel, dim3((N + warps - 1) / warps), dim3(warps * 32), 0, stream, logits, ld, correction, E,
+                       top, ids, wts, N, scale);
 }
 
 // tokens i32 [n_tokens], rows i32 [N] or null (then N == n_tokens), table i32 [V, top] -> ids i32 [N, top], wts f32 [N, top]
@@ -299,6 +399,25 @@ IIAN_API int iian_moe_combine_add(const void * ys, const int * pos, const float 
     return IIAN_ERR_DTYPE;
 }
 
+// wts: f32 [N, top]; h: A [N, W], the rows choices without an expert (pos < 0) pass on; add: A [N, W] or null (it may be `out`),
+// times sigmoid(add_gate[t * ld_gate]) if given.
+IIAN_API int iian_moe_combine_mixed(const void * ys, const int * pos, const float * wts, const void * h, const void * add,
+                                    const float * add_gate, long long ld_gate, void * out, int act_dtype, int N, int W, int top,
+                                    cudaStream_t stream) {
+    if (N <= 0) return IIAN_OK;
+    if (act_dtype != IIAN_F32 && act_dtype != IIAN_BF16) return IIAN_ERR_DTYPE;
+    const int V = act_dtype == IIAN_F32 ? 4 : 8;
+    const bool vec = W % V == 0 && (((uintptr_t) ys | (uintptr_t) h | (uintptr_t) add | (uintptr_t) out) & 15) == 0;
+    const int cols = vec ? W / V : W;
+    const int threads = cols >= 256 ? 256 : (cols + 31) / 32 * 32;
+    const dim3 grid(N, N >= 1024 ? 1 : min((cols + threads - 1) / threads, 8));
+#define IIAN_MIX(A, V) iian_launch(moe_combine_mixed_kernel<A, V>, grid, dim3(threads), 0, stream, (const A *) ys, pos, wts, (const A *) h, \
+                                   (A *) out, W, top, (const A *) add, add_gate, ld_gate)
+    if (act_dtype == IIAN_F32) return vec ? IIAN_MIX(float, 4) : IIAN_MIX(float, 1);
+    return vec ? IIAN_MIX(__nv_bfloat16, 8) : IIAN_MIX(__nv_bfloat16, 1);
+#undef IIAN_MIX
+}
+
 IIAN_API int iian_moe_combine_weighted(const void * ys, const int * pos, const float * wts, void * out, int act_dtype, int N, int W,
                                        int top, cudaStream_t stream) {
     return iian_moe_combine_add(ys, pos, wts, nullptr, out, act_dtype, N, W, top, stream);
@@ -308,7 +427,8 @@ IIAN_API int iian_moe_combine(const void * ys, const int * pos, void * out, int 
     return iian_moe_combine_weighted(ys, pos, nullptr, out, act_dtype, N, W, top, stream);
 }
 
-// x [M, K] sorted by expert; w (and w2, for the gated form) [E, n_out, K]; out [M, n_out]; act: 0 silu, 1 gelu (tanh).
+// x [M, K] sorted by expert; w (and w2, for the gated form) [E, n_out, K]; out [M, n_out]; act: 0 silu, 1 gelu (tanh); without
+// w2: 3 = max(z, 0)^2, anything else = the product as it is.
 // w2 == w: the gated form over blocks [E, 2 n_out, K] that hold both matrices interleaved in groups of 8 rows.
 // The plan's row tiles must be of iian_moe_tile_rows() rows.  act 2 (clamped, see moe_gated) takes `limit`.
 IIAN_API int iian_moe_grouped_gemm_act(const void * x, const void * w, const void * w2, void * out, const int * offsets,

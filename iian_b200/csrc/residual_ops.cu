@@ -6,6 +6,7 @@
 //   gelu_mul_table        out[r, :] = gelu_tanh(g[r, :]) * table[token(r), off : off + n]            token(r) = tokens[rows ? rows[r] : r]
 //   rms_norm_rows         out = x / sqrt(mean(x^2) + eps) * w for rows x of a wider matrix (row stride ld)
 //   xielu                 z > 0: softplus(p) z^2 + z / 2;  else (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2
+//   relu2                 max(z, 0)^2
 //   tanh_cap              z <- cap * tanh(z / cap), in place
 //   normed_add_rms_norm   x += y / sqrt(mean(y^2) + eps_y) * u [+ e]  (a sub-layer output that passes a norm of its own before
 //                         it joins the stream; e: a second float32 addend);  out = x / sqrt(mean(x^2) + eps) * w    (each optional)
@@ -258,6 +259,36 @@ __global__ void xielu_vec_kernel(const A * __restrict__ x, const float * __restr
     }
 }
 
+// max(z, 0)^2: scalar, or four entries at a time as the kernel above
+template <typename A>
+__global__ void relu2_kernel(const A * x, A * out, long long total) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const long long e = (long long) blockIdx.x * blockDim.x + threadIdx.x;
+    if (e >= total) return;
+    const float z = fmaxf(to_f32(x[e]), 0.0f);
+    out[e] = from_f32<A>(z * z);
+}
+
+template <typename A>
+__global__ void relu2_vec_kernel(const A * x, A * out, long long quads) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const long long e0 = (long long) blockIdx.x * blockDim.x * kXieluQuads + threadIdx.x;
+    float4 z[kXieluQuads];
+#pragma unroll
+    for (int i = 0; i < kXieluQuads; i++) {
+        const long long e = e0 + (long long) i * blockDim.x;
+        if (e < quads) z[i] = load4(x + 4 * e);
+    }
+#pragma unroll
+    for (int i = 0; i < kXieluQuads; i++) {
+        const long long e = e0 + (long long) i * blockDim.x;
+        z[i].x = fmaxf(z[i].x, 0.0f); z[i].y = fmaxf(z[i].y, 0.0f); z[i].z = fmaxf(z[i].z, 0.0f); z[i].w = fmaxf(z[i].w, 0.0f);
+        if (e < quads) store4(out + 4 * e, make_float4(z[i].x * z[i].x, z[i].y * z[i].y, z[i].z * z[i].z, z[i].w * z[i].w));
+    }
+}
+
 __global__ void tanh_cap_kernel(float * __restrict__ x, float cap, long long total) {
     pdl_wait();
     pdl_launch_dependents();
@@ -468,6 +499,23 @@ IIAN_API int iian_xielu(const void * x, const float * pq, void * out, int act_dt
         return iian_launch(xielu_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream, (const __nv_bfloat16 *) x, pq,
                            (__nv_bfloat16 *) out, total);
     return IIAN_ERR_DTYPE;
+}
+
+// x and out may be the same rows
+IIAN_API int iian_relu2(const void * x, void * out, int act_dtype, long long total, cudaStream_t stream) {
+    if (total <= 0) return IIAN_OK;
+    if (act_dtype != IIAN_F32 && act_dtype != IIAN_BF16) return IIAN_ERR_DTYPE;
+    const int threads = 256;
+    const int eb = act_dtype == IIAN_F32 ? 4 : 2;
+    if (total % 4 == 0 && (uintptr_t) x % (4 * eb) == 0 && (uintptr_t) out % (4 * eb) == 0) {
+        const long long quads = total / 4;
+        const unsigned vb = (unsigned) ((quads + (long long) threads * kXieluQuads - 1) / ((long long) threads * kXieluQuads));
+        if (act_dtype == IIAN_F32) return iian_launch(relu2_vec_kernel<float>, dim3(vb), dim3(threads), 0, stream, (const float *) x, (float *) out, quads);
+        return iian_launch(relu2_vec_kernel<__nv_bfloat16>, dim3(vb), dim3(threads), 0, stream, (const __nv_bfloat16 *) x, (__nv_bfloat16 *) out, quads);
+    }
+    const unsigned blocks = (unsigned) ((total + threads - 1) / threads);
+    if (act_dtype == IIAN_F32) return iian_launch(relu2_kernel<float>, dim3(blocks), dim3(threads), 0, stream, (const float *) x, (float *) out, total);
+    return iian_launch(relu2_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream, (const __nv_bfloat16 *) x, (__nv_bfloat16 *) out, total);
 }
 
 IIAN_API int iian_tanh_cap(float * x, float cap, long long total, cudaStream_t stream) {

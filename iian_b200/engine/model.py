@@ -109,6 +109,9 @@ class Model:
         self.weight_bytes = sum(t.numel() * t.element_size() for t in loaded.values())
         for _, part in scoped:
             part.bind(per_part.get(id(part), {}))
+        for block in self.blocks:
+            if hasattr(block, "bound"):
+                block.bound()
         if getattr(self.head, "tied", False):
             self.head.tie(self.embedding.weight)
         self.vocab_size = self.spec.vocab_size
@@ -203,7 +206,9 @@ class Model:
             select = ctx.out_rows if idx == len(order) - 1 else None
             block = self.blocks[call.layer]
             if call.before is not None:
-                residual, delta = self.stream_parts[call.before].forward(residual, delta, ctx)
+                part = self.stream_parts[call.before]
+                turn = {"turn": call.turn} if getattr(part, "wants_turn", False) else {}
+                residual, delta = part.forward(residual, delta, ctx, **turn)
             extra = {}
             if idx + 1 < len(order) and getattr(block, "accepts_next_norm", False):
                 # the block after this one: its first norm may ride in this block's last product

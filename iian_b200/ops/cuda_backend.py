@@ -909,7 +909,7 @@ class CudaKernels:
                   terms[0].shape[0], 1 if last_is_selected else 0, _cuda(out, "mix out", torch.float32), _cuda(out_act, "mix out"),
                   _code(out_act, "mix out") if out_act is not None else F32, r, h, _stream()), "depth_mix")
 
-    ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
+    ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2, "relu2": 3}
 
     def gated_act(self, gate_up: torch.Tensor, out: torch.Tensor, interleave: int, activation: str, limit: float = 0.0) -> None:
         """``out = act(gate) * up`` for rows ``[gate | up]`` (or interleaved in groups of 8); ``gate_up`` may be a column slice.
@@ -1089,16 +1089,16 @@ class CudaKernels:
 
     def moe_tcgen05_ok(self, dtype: torch.dtype, hidden: int, inter: int, activation: str) -> bool:
         """Whether both grouped products of an expert feed-forward can run on the tcgen05 kernel: bfloat16, rows of 16
-        bytes' multiples for TMA, gate and up interleaved in groups of 8 (SiLU rides in the product's epilogue; the clamped
-        activation is a pass of its own between the two products)."""
+        bytes' multiples for TMA, gate and up interleaved in groups of 8 (SiLU, and the squared positive part of experts without
+        a gate, ride in the product's epilogue; the clamped activation is a pass of its own between the two products)."""
         return (self.MOE_TCGEN05 and not self.LIBRARY_GEMM_ONLY and dtype == torch.bfloat16
-                and activation in ("silu", "clamped_swish") and hidden % 8 == 0 and inter % 8 == 0)
+                and activation in ("silu", "clamped_swish", "relu2") and hidden % 8 == 0 and inter % 8 == 0)
 
     def moe_grouped_gemm_tc(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: torch.Tensor, tiles: torch.Tensor,
-                            gated: bool) -> None:
+                            gated: bool, relu2: bool = False) -> None:
         """Rows of ``x`` sorted by expert times that expert's block of ``w`` [E, n, K] on tcgen05; ``gated``: the block's
-        rows are gate and up interleaved in groups of 8 and ``out`` [M, n / 2] = silu(gate) * up.  The plan's row tiles
-        are of 128 rows."""
+        rows are gate and up interleaved in groups of 8 and ``out`` [M, n / 2] = silu(gate) * up; ``relu2`` (not gated): ``out``
+        = max(product, 0)^2.  The plan's row tiles are of 128 rows."""
         m, k = x.shape
         e, n = w.shape[0], w.shape[1]
         if w.shape[2] != k or out.shape != (m, n // 2 if gated else n) or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 \
@@ -1110,7 +1110,7 @@ class CudaKernels:
         fn = _fn("gemm_tcgen05", "iian_gemm_tcgen05_grouped",
                  [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
                   c_void_p])
-        _check(fn(_cuda(x, "moe rows"), _cuda(w, "expert weights"), _cuda(out, "moe out"), BF16, m, n, e, k, 1 if gated else 0, bn,
+        _check(fn(_cuda(x, "moe rows"), _cuda(w, "expert weights"), _cuda(out, "moe out"), BF16, m, n, e, k, 1 if gated else 3 if relu2 else 0, bn,
                   status, _cuda(tiles, "tiles", torch.int32), _cuda(offsets, "offsets", torch.int32), (tiles.numel() - 1) // 2,
                   _stream()), "gemm_tcgen05_grouped")
 
@@ -1146,8 +1146,8 @@ class CudaKernels:
 
     def moe_grouped_gemm(self, x: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor], out: torch.Tensor,
                          offsets: torch.Tensor, tiles: torch.Tensor, activation: str = "silu", limit: float = 0.0) -> None:
-        """Rows of ``x`` sorted by expert times that expert's block of ``w`` [E, n_out, K]; with ``w2`` the gated form
-        ``act(x . w) * (x . w2)``; with ``w2 is w`` the blocks are [E, 2 n_out, K] and hold both matrices interleaved in
+        """Rows of ``x`` sorted by expert times that expert's block of ``w`` [E, n_out, K] (``relu2``: its positive part squared);
+        with ``w2`` the gated form ``act(x . w) * (x . w2)``; with ``w2 is w`` the blocks are [E, 2 n_out, K] and hold both matrices interleaved in
         groups of 8 rows."""
         m, k = x.shape
         n_out = w.shape[1] // 2 if w2 is w else w.shape[1]
@@ -1410,6 +1410,13 @@ class CudaKernels:
         _check(fn(_cuda(x, "xielu in"), _cuda(pq, "xielu numbers", torch.float32), _cuda(out, "xielu out"), _code(x, "xielu in"),
                   x.numel(), _stream()), "xielu")
 
+    def relu2(self, x: torch.Tensor, out: torch.Tensor) -> None:
+        """``out = max(x, 0)^2`` element by element; ``out`` may be ``x``."""
+        if out.shape != x.shape or out.dtype != x.dtype:
+            raise KernelError("relu2: out must match x")
+        fn = _fn("residual_ops", "iian_relu2", [c_void_p, c_void_p, c_int, c_longlong, c_void_p])
+        _check(fn(_cuda(x, "relu2 in"), _cuda(out, "relu2 out"), _code(x, "relu2 in"), x.numel(), _stream()), "relu2")
+
     def tanh_cap(self, x: torch.Tensor, cap: float) -> None:
         """``x <- cap * tanh(x / cap)`` in place (float32)."""
         fn = _fn("residual_ops", "iian_tanh_cap", [c_void_p, c_float, c_longlong, c_void_p])
@@ -1553,6 +1560,32 @@ class CudaKernels:
                   post_eps, _cuda(extra, "second addend", torch.float32), _cuda(weight, "norm weight", torch.float32),
                   _cuda(out, "norm out"), _code(act, "norm out"), n, h, eps, _stream()), "normed_add_rms_norm")
 
+    # ---- a norm by tanh, with a sub-layer output that passes such a norm before it joins the stream (csrc/tanh_norm.cu) -------
+    def tanh_add_tanh(self, residual: torch.Tensor, y: Optional[torch.Tensor], alpha_y: float, weight_y: Optional[torch.Tensor],
+                      bias_y: Optional[torch.Tensor], row: Optional[torch.Tensor], alpha: float, weight: Optional[torch.Tensor],
+                      bias: Optional[torch.Tensor], out: Optional[torch.Tensor]) -> None:
+        """``residual += weight_y tanh(alpha_y y) + bias_y`` (``y`` as it is without ``weight_y``) ``+ row`` (a float32 vector that
+        every row gets), in place; ``out`` receives ``weight tanh(alpha residual) + bias``.  Each of ``y``, ``row``, ``out`` may be
+        None."""
+        n, h = residual.shape
+        act = out if out is not None else y if y is not None else residual
+        for name, t in (("y", y), ("out", out)):
+            if t is not None and (t.shape != residual.shape or t.dtype != act.dtype):
+                raise KernelError(f"tanh_add_tanh: {name} {tuple(t.shape)} {t.dtype} does not match the stream {tuple(residual.shape)}")
+        for name, t in (("weight_y", weight_y), ("bias_y", bias_y), ("row", row), ("weight", weight), ("bias", bias)):
+            if t is not None and t.numel() != h:
+                raise KernelError(f"tanh_add_tanh: {name} does not match the stream")
+        f32 = torch.float32
+        fn = _fn("tanh_norm", "iian_tanh_add_tanh", [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
+                                                     c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+        _check(fn(_cuda(residual, "residual", f32), _cuda(y, "addend"), alpha_y, _cuda(weight_y, "addend norm weight", f32),
+                  _cuda(bias_y, "addend norm bias", f32), _cuda(row, "row", f32), alpha, _cuda(weight, "norm weight", f32),
+                  _cuda(bias, "norm bias", f32), _cuda(out, "norm out"), _code(act, "norm out"), n, h, _stream()), "tanh_add_tanh")
+
+    def add_row(self, residual: torch.Tensor, row: torch.Tensor) -> None:
+        """``residual += row`` for every row of the float32 stream."""
+        self.tanh_add_tanh(residual, None, 0.0, None, None, row, 0.0, None, None, None)
+
     def weighted_sum2(self, x: torch.Tensor, a: float, y: torch.Tensor, b: float, out: torch.Tensor) -> None:
         """``out = a x + b y`` element by element (one dtype, one shape)."""
         if x.shape != y.shape or out.shape != x.shape or x.dtype != y.dtype or out.dtype != x.dtype:
@@ -1654,6 +1687,53 @@ class CudaKernels:
                   n, num_heads, num_kv_heads, k_dim, v_dim, k_cache.shape[2], k_cache.shape[0], scale, window or 0, keep_first,
                   _cuda(sink, "sink", torch.float32), gp, ld_g, 1 if gate_per_head else 0, _stream()), "window_attention")
 
+    # ---- heads as the difference of two softmax maps over the same values (csrc/difference_attention.cu) ------------------------
+    def rotate_pairs_store(self, proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: torch.Tensor,
+                           k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], table: Optional[torch.Tensor],
+                           slots: Optional[torch.Tensor], *, num_heads: int, num_kv_heads: int, maps: int, k_dim: int, v_dim: int,
+                           rot_dim: int) -> None:
+        """Per token: rotate the first ``rot_dim`` entries of every sub-head of ``k_dim`` of q (``num_heads`` of them) and of k
+        (``num_kv_heads`` x ``maps``), entries 2i and 2i + 1 by the table's angle i; q to ``q_out`` [N, num_heads * k_dim], k (the
+        maps of a head side by side) and the values as projected to the token's cache cells (``k_cache`` None: q only)."""
+        n = proj.shape[0]
+        pp, ld = self._rows(proj, "projections")
+        if q_out.shape != (n, num_heads * k_dim) or q_out.dtype != proj.dtype:
+            raise KernelError("rotate_pairs_store: q_out must be [N, heads * k_dim] in the projections' dtype")
+        if k_cache is not None and (k_cache.shape[1] != num_kv_heads or k_cache.shape[3] != maps * k_dim or v_cache.shape[3] != v_dim
+                                    or k_cache.shape[:3] != v_cache.shape[:3] or k_cache.dtype != proj.dtype or slots.numel() != n):
+            raise KernelError(f"rotate_pairs_store: caches {tuple(k_cache.shape)} / {tuple(v_cache.shape)} do not fit")
+        if rot_dim and (table is None or table.shape != (n, rot_dim // 2, 2) or table.dtype != torch.float32):
+            raise KernelError("rotate_pairs_store: the rotation table must be float32 [N, rot_dim / 2, 2]")
+        fn = _fn("difference_attention", "iian_rotate_pairs_store",
+                 [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                  c_int, c_int, c_int, c_int, c_int, c_longlong, c_void_p])
+        page = k_cache.shape[2] if k_cache is not None else 1
+        cells = k_cache.shape[0] * k_cache.shape[2] if k_cache is not None else 0
+        _check(fn(pp, ld, q_off, k_off, v_off, _cuda(q_out, "queries"), _cuda(k_cache, "key cache"), _cuda(v_cache, "value cache"),
+                  _cuda(table if rot_dim else None, "rotary table"), _cuda(slots, "slots", torch.int32), _code(proj, "projections"), n,
+                  num_heads, num_kv_heads, maps, k_dim, v_dim, rot_dim, page, cells, _stream()), "rotate_pairs_store")
+
+    def difference_attention(self, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, meta, *,
+                             num_heads: int, num_kv_heads: int, k_dim: int, v_dim: int, scale: float, softcap: Optional[float],
+                             lam: float, factor: float, eps: float) -> None:
+        """``q`` [N, heads * 2 * k_dim] -> ``out`` [N, heads * v_dim]: per head the two maps' softmax (scores ``q . k * scale``,
+        then ``softcap tanh(./softcap)``; causal) over the cached keys, ``o = a1 - lam a2`` of the values both share, ``o``
+        divided by its root mean square over the head, times ``factor``."""
+        n = q.shape[0]
+        if q.shape[1] != num_heads * 2 * k_dim or out.shape != (n, num_heads * v_dim) or out.dtype != q.dtype \
+                or k_cache.dtype != q.dtype or k_cache.shape[3] != 2 * k_dim or v_cache.shape[3] != v_dim \
+                or k_cache.shape[1] != num_kv_heads:
+            raise KernelError(f"difference_attention: q {tuple(q.shape)}, out {tuple(out.shape)}, cache {tuple(k_cache.shape)} do not fit")
+        bt = meta.block_table
+        fn = _fn("difference_attention", "iian_difference_attention",
+                 [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                  c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_float, c_void_p])
+        _check(fn(_cuda(q, "queries"), _cuda(k_cache, "key cache"), _cuda(v_cache, "value cache"), _cuda(out, "attention out"),
+                  _cuda(meta.positions, "positions", torch.int32), _cuda(meta.seq_of_token, "seq_of_token", torch.int32),
+                  _cuda(bt, "block table", torch.int32), bt.shape[1], _cuda(meta.ctx_len, "ctx_len", torch.int32), _code(q, "queries"),
+                  n, num_heads, num_kv_heads, k_dim, v_dim, k_cache.shape[2], k_cache.shape[0], scale, softcap or 0.0, lam, factor,
+                  eps, _stream()), "difference_attention")
+
     # ---- linear attention with a decay: a matrix state per head (csrc/decay_scan.cu) -----------------------------------------
     def decay_scan(self, proj: torch.Tensor, q_off: int, k_off: int, v_off: int, state: torch.Tensor, cu_q: torch.Tensor,
                    state_slots: torch.Tensor, out: torch.Tensor, *, num_heads: int, dim: int, v_dim: int, activation: Optional[str],
@@ -1700,6 +1780,37 @@ class CudaKernels:
         _check(fn(lp, ld, _cuda(bias, "router bias", torch.float32), e, top, _cuda(ids, "expert ids", torch.int32),
                   _cuda(weights, "expert weights", torch.float32), n, _stream()), "moe_route_softmax")
 
+    def moe_route_corrected(self, logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, ids: torch.Tensor,
+                            weights: torch.Tensor, scale: float) -> None:
+        """Scores ``s = softmax(logits)`` (float32, may be a column slice); the ``top`` outputs with the largest ``s + correction``
+        (ties to the lower index), each weighing ``scale * s``."""
+        n, e = logits.shape
+        if logits.dtype != torch.float32 or ids.shape != (n, top) or weights.shape != (n, top) \
+                or (correction is not None and correction.numel() != e):
+            raise KernelError("moe_route_corrected: logits float32 [N, E]; correction [E]; ids / weights [N, top]")
+        lp, ld = self._rows(logits, "router logits")
+        fn = _fn("moe", "iian_moe_route_corrected", [c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
+                                                     c_void_p])
+        _check(fn(lp, ld, _cuda(correction, "choice correction", torch.float32), e, top, _cuda(ids, "expert ids", torch.int32),
+                  _cuda(weights, "expert weights", torch.float32), scale, n, _stream()), "moe_route_corrected")
+
+    def moe_combine_mixed(self, ys: torch.Tensor, pos: torch.Tensor, weights: torch.Tensor, h: torch.Tensor, out: torch.Tensor, top: int,
+                          add: Optional[torch.Tensor], add_gate: Optional[torch.Tensor]) -> None:
+        """``out[t] = sum_k weights[t, k] * (ys[pos[t, k]] or, where pos < 0, h[t]) + sigmoid(add_gate[t]) * add[t]`` (k ascending,
+        float32; ``add_gate`` None: factor 1; ``add`` None: nothing); ``add_gate`` float32 [N, 1], may be a column slice;
+        ``add`` may be ``out`` itself."""
+        n, w = out.shape
+        if ys.shape != (n * top, w) or ys.dtype != out.dtype or h.shape != out.shape or h.dtype != out.dtype \
+                or weights.numel() != n * top or (add is not None and (add.shape != out.shape or add.dtype != out.dtype)) \
+                or (add_gate is not None and (add_gate.shape != (n, 1) or add_gate.dtype != torch.float32)):
+            raise KernelError("moe_combine_mixed: ys [N * top, W], h and add [N, W] in the dtype of out, add_gate float32 [N, 1]")
+        gp, ld = (add_gate.data_ptr(), add_gate.stride(0)) if add_gate is not None else (0, 0)
+        fn = _fn("moe", "iian_moe_combine_mixed", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int,
+                                                   c_int, c_int, c_int, c_void_p])
+        _check(fn(_cuda(ys, "moe out rows"), _cuda(pos, "pos", torch.int32), _cuda(weights, "expert weights", torch.float32),
+                  _cuda(h, "moe in"), _cuda(add, "addend"), gp, ld, _cuda(out, "moe out"), _code(out, "moe out"), n, w, top, _stream()),
+               "moe_combine_mixed")
+
     def moe_combine_add(self, ys: torch.Tensor, pos: torch.Tensor, out: torch.Tensor, top: int, weights: Optional[torch.Tensor],
                         add: torch.Tensor) -> None:
         """``out[t] = sum_k weights[t, k] * ys[pos[t, k]] + add[t]`` (k ascending, float32); ``add`` may be ``out`` itself."""
@@ -1720,10 +1831,11 @@ class CudaKernels:
 
     def delta_rule(self, proj: torch.Tensor, col_off: int, b_off: int, z: torch.Tensor, taps: torch.Tensor, a_log: torch.Tensor,
                    dt_bias: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, *, num_heads: int, num_kv_heads: int, dim: int,
-                   v_dim: int) -> None:
+                   v_dim: int, b_pre: Optional[torch.Tensor] = None) -> None:
         """The recurrence over this step's tokens of every sequence.  ``proj`` rows hold the convolution's inputs q | k | v at
-        column ``col_off`` and the write strengths' pre-activations at ``b_off``; ``z`` float32 [N, heads * dim] the decays'
-        pre-activations without bias; ``taps`` float32 [channels, taps]; ``state`` float32 [slots, state floats];
+        column ``col_off`` and the write strengths' pre-activations at ``b_off`` (or ``b_pre`` float32 [N, heads] holds them);
+        ``z`` float32 [N, heads * dim] (a decay per key channel) or [N, heads] (one per head) the decays' pre-activations
+        without bias; ``z`` and ``b_pre`` may be column slices of one matrix; ``taps`` float32 [channels, taps]; ``state`` float32 [slots, state floats];
         ``out`` float32 [N, heads * v_dim] receives ``S^T q`` per head.  Two launches: per-token preparation, then the scan."""
         n = proj.shape[0]
         h, g, d, v = num_heads, num_kv_heads, dim, v_dim
@@ -1731,7 +1843,12 @@ class CudaKernels:
         n_taps = taps.shape[1]
         pp, ld = self._rows(proj, "projections")
         s = ctx.cu_q.numel() - 1
-        if z.shape != (n, h * d) or taps.shape[0] != channels or a_log.numel() != h or dt_bias.numel() != h * d \
+        per_head = z.shape == (n, h) and d != 1
+        zp, ld_z = self._rows(z, "decay pre-activations")
+        bp, ld_b = self._rows(b_pre, "write strengths") if b_pre is not None else (0, ld_z)
+        if z.dtype != torch.float32 or (b_pre is not None and (b_pre.shape != (n, h) or b_pre.dtype != torch.float32 or ld_b != ld_z)):
+            raise KernelError("delta_rule: z and b_pre are float32 with one row stride")
+        if (not per_head and z.shape != (n, h * d)) or taps.shape[0] != channels or a_log.numel() != h or dt_bias.numel() != z.shape[1] \
                 or out.shape != (n, h * v) or state.dim() != 2 or state.shape[1] != self.delta_state_floats(h, g, d, v, n_taps) \
                 or ctx.state_slots.numel() != s:
             raise KernelError("delta_rule: shapes do not fit")
@@ -1740,24 +1857,25 @@ class CudaKernels:
         kn = ctx.buf("delta_k", (n, g * d), f32)
         vv = ctx.buf("delta_v", (n, h * v), f32)
         beta = ctx.buf("delta_beta", (n, h), f32)
-        decay = ctx.buf("delta_decay", (n, h * d), f32)
+        decay = ctx.buf("delta_decay", (n, z.shape[1]), f32)
         qk = ctx.buf("delta_qk", (n, g), f32)
         code = _code(proj, "projections")
         fn = _fn("delta_rule", "iian_delta_prep",
-                 [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong,
-                  c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                  c_int, c_void_p])
-        _check(fn(pp, ld, col_off, b_off, code, _cuda(z, "decay pre-activations", f32), _cuda(taps, "taps", f32), n_taps,
+                 [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_void_p, c_void_p,
+                  c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                  c_int, c_int, c_int, c_int, c_void_p])
+        _check(fn(pp, ld, col_off, b_off, code, bp, zp, ld_z, 1 if per_head else 0, _cuda(taps, "taps", f32), n_taps,
                   _cuda(a_log, "A_log", f32), _cuda(dt_bias, "dt_bias", f32), _cuda(state, "state", f32), state.shape[1],
                   _cuda(ctx.seq_of_token, "seq_of_token", torch.int32), _cuda(ctx.cu_q, "cu_q", torch.int32),
                   _cuda(ctx.state_slots, "state slots", torch.int32), qn.data_ptr(), kn.data_ptr(), vv.data_ptr(), beta.data_ptr(),
                   decay.data_ptr(), qk.data_ptr(), n, h, g, d, v, _stream()), "delta_prep")
         fn = _fn("delta_rule", "iian_delta_scan",
                  [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int,
-                  c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+                  c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
         _check(fn(qn.data_ptr(), kn.data_ptr(), vv.data_ptr(), beta.data_ptr(), decay.data_ptr(), qk.data_ptr(), state.data_ptr(),
                   state.shape[1], pp, ld, col_off, code, n_taps, ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr(),
-                  _cuda(out, "delta out", f32), s, h, g, d, v, int(getattr(ctx, "max_q_len", 0) or 0), _stream()), "delta_scan")
+                  _cuda(out, "delta out", f32), s, h, g, d, v, int(getattr(ctx, "max_q_len", 0) or 0), 1 if per_head else 0, _stream()),
+               "delta_scan")
 
     # ---- routing by a table, weights on the experts' outputs (csrc/moe.cu) ------------------------------------------------------
     def moe_table_route(self, tokens: torch.Tensor, rows: Optional[torch.Tensor], table: torch.Tensor, num_experts: int,

@@ -193,6 +193,18 @@ class NormedAddend:
     extra: Optional[torch.Tensor] = None
 
 
+@dataclass
+class TanhAddend:
+    """The same for a post-norm that takes no statistics of the row: the stream becomes ``x + w tanh(alpha y) + b`` (a factor
+    per column behind the norm is already in ``w`` and ``b``) ``+ row``, ``row`` one float32 vector that every row gets
+    (optional).  The norm that runs next (``dynamic_tanh``) does it in its own kernel (``ops: tanh_add_tanh``)."""
+    y: torch.Tensor
+    alpha: float
+    weight: torch.Tensor
+    bias: torch.Tensor
+    row: Optional[torch.Tensor] = None
+
+
 class Norm(Part):
     def forward(self, residual: torch.Tensor, delta: Optional[torch.Tensor], ctx) -> torch.Tensor:  # pragma: no cover
         raise NotImplementedError
@@ -251,9 +263,12 @@ class StreamPart(Part):
 
     ``forward(residual, delta, ctx) -> (residual, delta)``: the float32 stream and what has not been added to it yet (None, a
     tensor, or a pair of tensors), as a block receives and returns them.  A part that reads what the embedding left says so
-    with ``needs_embedding_out``; the model then keeps that tensor untouched under ``ctx.step_cache["embedding_out"]``."""
+    with ``needs_embedding_out``; the model then keeps that tensor untouched under ``ctx.step_cache["embedding_out"]``.  A part
+    that acts differently in each run of a repeated stretch says so with ``wants_turn`` and is called with ``turn=`` the
+    number the run order gives (``LayerCall.turn``)."""
 
     needs_embedding_out = False
+    wants_turn = False
 
     def forward(self, residual: torch.Tensor, delta, ctx):  # pragma: no cover
         raise NotImplementedError

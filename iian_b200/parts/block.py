@@ -4,6 +4,7 @@ A block implements one arrangement (``LayerSpec.arrangement``) and is registered
 ``register_block``.  What the model asks of a block: ``__init__(spec, dtype, device)`` builds its parts from the
 slots of the ``LayerSpec`` it understands; ``parts()`` lists them with the slot names their tensors go under;
 ``cache_need()`` says what the cache of a call to this layer must hold (a ``KVNeed``, a ``StateNeed`` or None);
+``bound()`` (optional) is called once after all parts have their weights;
 ``forward(residual, delta, ctx, cache, writes_cache, select_rows)`` takes the float32 residual stream and the
 not-yet-added output of whatever ran before, and returns the same pair.
 
@@ -266,15 +267,39 @@ class ScaledResidualBlock:
         return residual, None
 
 
+class ColumnScale:
+    """A learned factor per column of a sub-layer's normalised output (a layer scale).  params: ``size``.  It has no kernel: the
+    arrangement takes it into the weight of the norm before it."""
+
+    graph_safe = True
+
+    def __init__(self, spec, dtype, device):
+        self.spec, self.dtype, self.device = spec, dtype, device
+        self.size = int(spec["size"])
+        self.weight = None
+
+    def tensors(self):
+        from ..weights.loader import TensorSpec
+        return {"weight": TensorSpec((self.size,), init="ones_jitter")}
+
+    def bind(self, tensors) -> None:
+        self.weight = tensors["weight"].to(torch.float32).contiguous()
+
+    def kernel_libraries(self):
+        return ()
+
+
 @register_block("sandwich_residual")
 class SandwichResidualBlock:
     """``x += nb1(mixer(n1 x))``; ``x += nb2(ffn(n2 x))``: a norm before AND after each sub-layer.
 
     Slots: ``mixer_norm``, ``mixer``; optionally ``feed_forward`` with ``feed_forward_norm``; in ``extra``
-    ``mixer_post_norm`` and (with a feed-forward) ``feed_forward_post_norm``, norms that offer ``as_addend`` (``rms_norm``).
-    A sub-layer's output is not added by a kernel of its own: wrapped as a ``NormedAddend`` it goes to the norm that runs
-    next, whose kernel normalises it, adds it to the float32 stream and normalises the stream (the block's last one is handed
-    on as ``delta``).  With ``select_rows`` (the run order's last entry) only the wanted rows go on after the mixer."""
+    ``mixer_post_norm`` and (with a feed-forward) ``feed_forward_post_norm``, norms that offer ``as_addend`` (``rms_norm``,
+    ``dynamic_tanh``), and optionally ``mixer_scale`` / ``feed_forward_scale`` (:class:`ColumnScale`): a factor per column
+    behind the post-norm, ``x += c * nb1(mixer(n1 x))``.
+    A sub-layer's output is not added by a kernel of its own: wrapped as a ``NormedAddend`` or a ``TanhAddend`` it goes to the
+    norm that runs next, whose kernel normalises it, adds it to the float32 stream and normalises the stream (the block's last
+    one is handed on as ``delta``); the factor is part of the post-norm's weight.  With ``select_rows`` (the run order's last entry) only the wanted rows go on after the mixer."""
 
     def __init__(self, spec: LayerSpec, dtype: torch.dtype, device: torch.device):
         need = ["mixer", "mixer_norm", "mixer_post_norm"]
@@ -295,14 +320,27 @@ class SandwichResidualBlock:
             self.feed_forward_post_norm = NORMS.build(spec.slot("feed_forward_post_norm"), dtype, device)
         for norm in (self.mixer_post_norm, self.feed_forward_post_norm):
             if norm is not None and not hasattr(norm, "as_addend"):
-                raise ValueError("arrangement sandwich_residual needs post-norms that can ride in the next norm's sum (rms_norm)")
+                raise ValueError("arrangement sandwich_residual needs post-norms that can ride in the next norm's sum "
+                                 "(rms_norm, dynamic_tanh)")
+        m, f = spec.slot("mixer_scale"), spec.slot("feed_forward_scale")
+        self.mixer_scale = ColumnScale(m, dtype, device) if m is not None else None
+        self.feed_forward_scale = ColumnScale(f, dtype, device) if f is not None and self.feed_forward is not None else None
 
     def parts(self):
         out = [("mixer_norm", self.mixer_norm), ("mixer", self.mixer), ("mixer_post_norm", self.mixer_post_norm)]
         if self.feed_forward is not None:
             out += [("feed_forward_norm", self.feed_forward_norm), ("feed_forward", self.feed_forward),
                     ("feed_forward_post_norm", self.feed_forward_post_norm)]
+        for name in ("mixer_scale", "feed_forward_scale"):
+            if getattr(self, name) is not None:
+                out.append((name, getattr(self, name)))
         return tuple(out)
+
+    def bound(self) -> None:
+        """Called once after every part has its weights: a factor per column behind a post-norm becomes part of that norm's weight."""
+        for scale, norm in ((self.mixer_scale, self.mixer_post_norm), (self.feed_forward_scale, self.feed_forward_post_norm)):
+            if scale is not None:
+                norm.absorb_factor(scale.weight)
 
     def cache_need(self):
         return self.mixer.cache_need()

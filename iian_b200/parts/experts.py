@@ -21,6 +21,14 @@ logits are taken and weighed by the softmax over those logits ALONE.  ``shared_i
 feed-forward of that width (tensors ``shared.gate / up / down``, same activation) that every token uses; its output is added
 to the experts' sum in the kernel that forms it.
 
+``score = "softmax"``: scores are the softmax over all router outputs, without a bias; the ``top`` outputs with the largest
+score plus ``correction`` (a number per output that only the choice sees) are taken and weighed by ``weight_scale`` times their
+score, not renormalised.  ``identity_experts``: the last so many router outputs have no expert behind them; a token that takes
+one gets its own input, times the weight: such choices get no row in the sorted rows, the kernel that sums the experts reads
+the input instead.  ``activation = "relu2"``: experts without a gate, ``Wdown max(Wup u, 0)^2``; the shared one has the same form.
+``shared_gate``: the shared expert's output is multiplied by ``sigmoid(w h)``, one number per token; its row ``shared.sg``
+rides under the router's in the product with float32 output.
+
 ``stack_rows`` puts further rows that read the same input (a gate of the residual) under the router's, so that one
 product with float32 output serves both.
 """
@@ -38,8 +46,9 @@ from .base import FeedForward, register_feed_forward
 @register_feed_forward("routed_experts")
 class RoutedExperts(FeedForward):
     """params: ``hidden_size``, ``num_experts``, ``top``, ``intermediate_size`` (of one expert), ``activation``
-    (``silu`` | ``gelu_tanh`` | ``clamped_swish`` with ``limit``), ``score`` (``sigmoid`` | ``table`` with ``vocab_size``),
-    ``weight_on`` (``input`` | ``output``)."""
+    (``silu`` | ``gelu_tanh`` | ``clamped_swish`` with ``limit`` | ``relu2``), ``score`` (``sigmoid`` | ``softmax_top`` | ``softmax``
+    with ``weight_scale`` and ``identity_experts`` | ``table`` with ``vocab_size``), ``weight_on`` (``input`` | ``output``),
+    ``shared_intermediate_size`` with ``shared_gate``."""
 
     SWISH_ALPHA = 1.702         # fixed by the clamped activation (also in the kernels)
 
@@ -51,30 +60,46 @@ class RoutedExperts(FeedForward):
         self.top = int(p["top"])
         self.inter = int(p["intermediate_size"])
         self.activation = p.get("activation", "silu")
-        if self.activation not in ("silu", "gelu_tanh", "clamped_swish"):
+        if self.activation not in ("silu", "gelu_tanh", "clamped_swish", "relu2"):
             raise ValueError(f"routed_experts: activation '{self.activation}' has no kernel")
         self.limit = float(p.get("limit", 0.0))
         if self.activation == "clamped_swish" and self.limit <= 0:
             raise ValueError("routed_experts: the clamped activation needs a positive limit")
         self.score = p.get("score", "sigmoid")
         self.weight_on = p.get("weight_on", "input")
-        if self.score not in ("sigmoid", "softmax_top", "table") or self.weight_on not in ("input", "output"):
-            raise ValueError("routed_experts: score is 'sigmoid', 'softmax_top' or 'table', weight_on 'input' or 'output'")
+        if self.score not in ("sigmoid", "softmax_top", "softmax", "table") or self.weight_on not in ("input", "output"):
+            raise ValueError("routed_experts: score is 'sigmoid', 'softmax_top', 'softmax' or 'table', weight_on 'input' or 'output'")
+        self.identity = int(p.get("identity_experts", 0) or 0)
+        self.weight_scale = float(p.get("weight_scale", 1.0))
+        if (self.identity or self.weight_scale != 1.0) and self.score != "softmax":
+            raise ValueError("routed_experts: identity_experts and weight_scale come with score 'softmax'")
+        if self.score == "softmax" and self.weight_on != "output":
+            raise ValueError("routed_experts: with score 'softmax' the weight is on the output")
+        self.outputs = self.experts + self.identity         # of the router
+        self.correction = None
         self.shared_inter = int(p.get("shared_intermediate_size", 0) or 0)
         self.shared = None
         if self.shared_inter:
-            if self.activation not in ("silu", "gelu_tanh"):
-                raise ValueError("routed_experts: the shared expert takes silu or gelu_tanh")
+            if self.activation not in ("silu", "gelu_tanh", "relu2"):
+                raise ValueError("routed_experts: the shared expert takes silu, gelu_tanh or relu2")
             from ..config.spec import PartSpec
-            from .mlp import GatedMLP
-            self.shared = GatedMLP(PartSpec("gated_mlp", {"hidden_size": self.hidden, "intermediate_size": self.shared_inter,
-                                                          "activation": self.activation,
-                                                          "names": ("shared.gate", "shared.up", "shared.down")}), dtype, device)
+            from .mlp import GatedMLP, PlainMLP
+            if self.activation == "relu2":
+                self.shared = PlainMLP(PartSpec("plain_mlp", {"hidden_size": self.hidden, "intermediate_size": self.shared_inter,
+                                                              "activation": "relu2",
+                                                              "names": ("shared.up", "shared.down", "shared.act")}), dtype, device)
+            else:
+                self.shared = GatedMLP(PartSpec("gated_mlp", {"hidden_size": self.hidden, "intermediate_size": self.shared_inter,
+                                                              "activation": self.activation,
+                                                              "names": ("shared.gate", "shared.up", "shared.down")}), dtype, device)
+        self.shared_gate = bool(p.get("shared_gate", False)) and self.shared is not None
+        if self.shared_gate and self.score != "softmax":
+            raise ValueError("routed_experts: shared_gate comes with score 'softmax'")
         self.router_bias = None
         self.vocab = int(p["vocab_size"]) if self.score == "table" else 0
         self.needs_tokens = self.score == "table"       # forward wants to know which token each row belongs to
-        if not 0 < self.top <= self.experts:
-            raise ValueError(f"routed_experts: top {self.top} of {self.experts} experts")
+        if not 0 < self.top <= self.outputs:
+            raise ValueError(f"routed_experts: top {self.top} of {self.outputs} experts")
         self.w_router = self.w_gate = self.w_up = self.w_down = self.w_gate_up = None
         self.extra_rows = None
         self.table = None
@@ -83,13 +108,18 @@ class RoutedExperts(FeedForward):
         if self.score == "table":
             t = {"table": TensorSpec((self.vocab, self.top), kind="int", init=f"distinct_rows:{self.experts}")}
         else:
-            t = {"router": TensorSpec((self.experts, self.hidden))}
+            t = {"router": TensorSpec((self.outputs, self.hidden))}
+            if self.score == "softmax":
+                t["correction"] = TensorSpec((self.outputs,), init="zeros_jitter")
+            if self.shared_gate:
+                t["shared.sg"] = TensorSpec((1, self.hidden))
             if self.score == "softmax_top":
                 t["router.b"] = TensorSpec((self.experts,))
         if self.shared is not None:
             t.update(self.shared.tensors())
         for e in range(self.experts):
-            t[f"e{e}.gate"] = TensorSpec((self.inter, self.hidden))
+            if self.activation != "relu2":
+                t[f"e{e}.gate"] = TensorSpec((self.inter, self.hidden))
             t[f"e{e}.up"] = TensorSpec((self.inter, self.hidden))
             t[f"e{e}.down"] = TensorSpec((self.hidden, self.inter))
         return t
@@ -102,8 +132,16 @@ class RoutedExperts(FeedForward):
             self.w_router = self._router.contiguous()
             if self.score == "softmax_top":
                 self.router_bias = tensors["router.b"].to(torch.float32).contiguous()
+            if self.score == "softmax":
+                self.correction = tensors["correction"].to(torch.float32).contiguous()
+            if self.shared_gate:
+                self.stack_rows(tensors["shared.sg"])
         if self.shared is not None:
             self.shared.bind({k: t for k, t in tensors.items() if k.startswith("shared.")})
+        if self.activation == "relu2":
+            self.w_up = torch.stack([tensors[f"e{e}.up"] for e in range(self.experts)]).contiguous()
+            self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(self.experts)]).contiguous()
+            return
         gate = torch.stack([tensors[f"e{e}.gate"] for e in range(self.experts)])
         up = torch.stack([tensors[f"e{e}.up"] for e in range(self.experts)])
         self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(self.experts)]).contiguous()
@@ -149,12 +187,14 @@ class RoutedExperts(FeedForward):
         else:
             logits = ctx.buf("router_logits", (n, self.w_router.shape[0]), torch.float32)
             k.linear(x, self.w_router, logits)
-            if self.score == "softmax_top":
+            if self.score == "softmax":
+                k.moe_route_corrected(logits[:, : self.outputs], self.correction, top, ids, wts, self.weight_scale)
+            elif self.score == "softmax_top":
                 k.moe_route_softmax(logits[:, :E], self.router_bias, top, ids, wts)
             else:
                 k.moe_route(logits[:, :E], top, ids, wts)
         on_input = self.weight_on == "input"
-        on_tc = (self.w_gate_up is not None and hasattr(k, "moe_tcgen05_ok")
+        on_tc = ((self.w_gate_up is not None or self.activation == "relu2") and hasattr(k, "moe_tcgen05_ok")
                  and k.moe_tcgen05_ok(self.dtype, self.hidden, self.inter, self.activation))
         tile_rows = k.MOE_TC_TILE_ROWS if on_tc else k.moe_tile_rows()
         max_tiles = k.moe_max_tiles(m, E, tile_rows)
@@ -166,7 +206,14 @@ class RoutedExperts(FeedForward):
         k.moe_scatter(x, pos, wts if on_input else None, xs, top)
         act = ctx.buf("expert_act", (m, self.inter), self.dtype)
         ys = ctx.buf("expert_out", (m, self.hidden), self.dtype)
-        if on_tc and self.activation != "silu":
+        if self.activation == "relu2":
+            if on_tc:
+                k.moe_grouped_gemm_tc(xs, self.w_up, act, offsets, tiles, gated=False, relu2=True)
+                k.moe_grouped_gemm_tc(act, self.w_down, ys, offsets, tiles, gated=False)
+            else:
+                k.moe_grouped_gemm(xs, self.w_up, None, act, offsets, tiles, "relu2")
+                k.moe_grouped_gemm(act, self.w_down, None, ys, offsets, tiles)
+        elif on_tc and self.activation != "silu":
             wide = ctx.buf("expert_gate_up", (m, 2 * self.inter), self.dtype)
             k.moe_grouped_gemm_tc(xs, self.w_gate_up, wide, offsets, tiles, gated=False)
             k.gated_act(wide, act, 8, self.activation, self.limit)
@@ -180,7 +227,11 @@ class RoutedExperts(FeedForward):
             else:
                 k.moe_grouped_gemm(xs, self.w_gate, self.w_up, act, offsets, tiles, self.activation, self.limit)
             k.moe_grouped_gemm(act, self.w_down, None, ys, offsets, tiles)
-        if self.shared is not None:
+        if self.score == "softmax":
+            add = self.shared.forward(x, ctx) if self.shared is not None else None        # lands in "ffn_out" and is summed in place
+            out = add if add is not None else ctx.buf("ffn_out", (n, self.hidden), self.dtype)
+            k.moe_combine_mixed(ys, pos, wts, x, out, top, add, logits[:, self.outputs: self.outputs + 1] if self.shared_gate else None)
+        elif self.shared is not None:
             out = self.shared.forward(x, ctx)                      # lands in "ffn_out"; the experts' sum is added onto it
             k.moe_combine_add(ys, pos, out, top, None if on_input else wts, out)
         else:

@@ -125,28 +125,31 @@ class PlainMLP(FeedForward):
     """A feed-forward without a gate: ``y = Wdown act(Wup h)``.
 
     params: ``hidden_size``, ``intermediate_size``, ``activation``: ``xielu`` (two learned numbers p, q in a tensor of
-    their own: ``z > 0: softplus(p) z^2 + z / 2``, else ``(1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2``); optional
-    ``names``: the local tensor names of (up, down, the activation's numbers)."""
+    their own: ``z > 0: softplus(p) z^2 + z / 2``, else ``(1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2``) or ``relu2``
+    (``max(z, 0)^2``, no tensor); optional ``names``: the local tensor names of (up, down, the activation's numbers)."""
 
     def __init__(self, spec, dtype, device):
         super().__init__(spec, dtype, device)
         self.hidden = int(spec["hidden_size"])
         self.inter = int(spec["intermediate_size"])
         act = spec.params.get("activation", "xielu")
-        if act != "xielu":
-            raise ValueError(f"plain_mlp: activation '{act}' has no kernel (xielu)")
+        if act not in ("xielu", "relu2"):
+            raise ValueError(f"plain_mlp: activation '{act}' has no kernel (xielu, relu2)")
         self.activation = act
         self.names = tuple(spec.params.get("names", ("up", "down", "act")))
         self.w_up = self.w_down = self.act_numbers = None
 
     def tensors(self) -> Dict[str, TensorSpec]:
-        return {self.names[0]: TensorSpec((self.inter, self.hidden)), self.names[1]: TensorSpec((self.hidden, self.inter)),
-                self.names[2]: TensorSpec((2,), init="zeros_jitter")}
+        t = {self.names[0]: TensorSpec((self.inter, self.hidden)), self.names[1]: TensorSpec((self.hidden, self.inter))}
+        if self.activation == "xielu":
+            t[self.names[2]] = TensorSpec((2,), init="zeros_jitter")
+        return t
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.w_up = tensors[self.names[0]].contiguous()
         self.w_down = tensors[self.names[1]].contiguous()
-        self.act_numbers = tensors[self.names[2]].to(torch.float32).contiguous()
+        if self.activation == "xielu":
+            self.act_numbers = tensors[self.names[2]].to(torch.float32).contiguous()
 
     def kernel_libraries(self):
         return ("residual_ops", "gemm_simt")
@@ -157,7 +160,10 @@ class PlainMLP(FeedForward):
         up = ctx.buf("ffn_up", (n, self.inter), self.dtype)
         k.linear(x, self.w_up, up)
         act = ctx.buf("ffn_act", (n, self.inter), self.dtype)
-        k.xielu(up, self.act_numbers, act)
+        if self.activation == "relu2":
+            k.relu2(up, act)
+        else:
+            k.xielu(up, self.act_numbers, act)
         out = ctx.buf("ffn_out", (n, self.hidden), self.dtype)
         k.linear(act, self.w_down, out)
         return out

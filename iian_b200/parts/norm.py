@@ -1,5 +1,5 @@
 """Norms.  RMSNorm, fused with the residual add that precedes it; LayerNorm with weight and bias, fused with the
-scaled and gated residual sum of a post-norm layer.
+scaled and gated residual sum of a post-norm layer; a norm by tanh that takes no statistics of the row.
 
 ``y = x * rsqrt(mean(x^2) + eps) * w``: normalise first, multiply by the weight second, no ``1 + w``
 and no bias (src/iian/graph.cpp:105-114).  The sum of squares and the residual sum are float32.
@@ -12,7 +12,7 @@ import torch
 
 from .. import ops
 from ..weights.loader import TensorSpec
-from .base import Norm, NormedAddend, register_norm
+from .base import Norm, NormedAddend, TanhAddend, register_norm
 
 
 @register_norm("rms_norm")
@@ -47,6 +47,10 @@ class RMSNorm(Norm):
 
     def as_addend(self, y: torch.Tensor) -> NormedAddend:
         return NormedAddend(y, self.weight, self.eps)
+
+    def absorb_factor(self, factor: torch.Tensor) -> None:
+        """A factor per column behind this norm becomes part of its weight."""
+        self.weight = (self.weight * factor).contiguous()
 
     def forward(self, residual: torch.Tensor, delta, ctx, delta_scale: float = 1.0) -> torch.Tensor:
         """``delta_scale``: the stream becomes ``x + delta_scale * delta`` (a design that adds its sub-layers' outputs with a
@@ -118,3 +122,53 @@ class LayerNorm(Norm):
         act = ctx.buf(f"stream_act_{name}", x.shape, self.dtype)
         ops.kernels().gated_add_layer_norm(x, sub, gate, gate_bias, self.weight, self.bias, alpha, self.eps, out, act)
         return out, act
+
+
+@register_norm("dynamic_tanh")
+class DynamicTanh(Norm):
+    """``y = w tanh(alpha x) + b``: element by element, no mean and no variance.  params: ``size``.  Tensors: ``weight`` and
+    ``bias`` per column, ``alpha`` one number.
+
+    ``delta`` may be a tensor, or a ``TanhAddend`` (a sub-layer output that passes a norm of this kind on its way into the
+    stream): the sum and both norms are one kernel.  ``as_addend(y)`` wraps a sub-layer output for THIS norm; a factor per
+    column behind it is taken into ``w`` and ``b`` (``absorb_factor``).  Everything is float32; only the rows it leaves for
+    the next product are in the activation dtype."""
+
+    def __init__(self, spec, dtype, device):
+        super().__init__(spec, dtype, device)
+        self.size = int(spec["size"])
+        self.alpha = 0.0
+        self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+
+    def tensors(self) -> Dict[str, TensorSpec]:
+        return {"weight": TensorSpec((self.size,), init="ones_jitter"), "alpha": TensorSpec((), init="ones_jitter"),
+                "bias": TensorSpec((self.size,), init="zeros_jitter")}
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.weight = tensors["weight"].to(torch.float32).contiguous()
+        self.bias = tensors["bias"].to(torch.float32).contiguous()
+        self.alpha = float(tensors["alpha"])
+
+    def kernel_libraries(self):
+        return ("tanh_norm",)
+
+    def as_addend(self, y: torch.Tensor) -> TanhAddend:
+        return TanhAddend(y, self.alpha, self.weight, self.bias)
+
+    def absorb_factor(self, factor: torch.Tensor) -> None:
+        self.weight = (self.weight * factor).contiguous()
+        self.bias = (self.bias * factor).contiguous()
+
+    def forward(self, residual: torch.Tensor, delta, ctx, delta_scale: float = 1.0) -> torch.Tensor:
+        if delta_scale != 1.0:
+            raise ValueError("dynamic_tanh: an addend takes no factor (a layer scale is part of the addend's norm)")
+        out = ctx.buf("normed", residual.shape, self.dtype)
+        if delta is not None and not isinstance(delta, (torch.Tensor, TanhAddend)):
+            raise ValueError("dynamic_tanh: the addend is a tensor or a TanhAddend")
+        if isinstance(delta, TanhAddend):
+            ops.kernels().tanh_add_tanh(residual, delta.y, delta.alpha, delta.weight, delta.bias, delta.row, self.alpha,
+                                        self.weight, self.bias, out)
+        else:
+            ops.kernels().tanh_add_tanh(residual, delta, 0.0, None, None, None, self.alpha, self.weight, self.bias, out)
+        return out

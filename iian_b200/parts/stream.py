@@ -3,6 +3,10 @@
 ``add_embedding``: ``x <- x + e`` with ``e`` what the embedding left.  Nothing is launched for it where the block before left
 a ``NormedAddend``: ``e`` rides as the second addend of the sum the next norm does anyway.
 
+``add_turn_vector``: ``x <- x + s_t`` with ``s_t`` a learned vector per run ``t`` of a stretch of layers that runs several
+times.  Nothing is launched for it where the block before left a ``TanhAddend``: the vector rides in the sum the next norm
+does anyway.
+
 ``reinject_embedding``: ``x <- W [x ; e]`` with ``e`` what the embedding left and ``W`` [hidden, 2 hidden] (the columns
 that meet ``x`` first).  A model that runs a stretch of its layers several times puts it before the first layer of every
 run, so that each run sees the input again.  The sum that is still owed to the stream (``delta``) is added while the
@@ -17,7 +21,7 @@ import torch
 
 from .. import ops
 from ..weights.loader import TensorSpec
-from .base import NormedAddend, StreamPart, register_stream_part
+from .base import NormedAddend, StreamPart, TanhAddend, register_stream_part
 
 
 @register_stream_part("reinject_embedding")
@@ -71,3 +75,33 @@ class EmbeddingAddition(StreamPart):
         if isinstance(delta, NormedAddend) and delta.extra is None:
             return residual, NormedAddend(delta.y, delta.weight, delta.eps, extra=e)
         raise ValueError("add_embedding: the block before must leave nothing or one normalised addend to the stream")
+
+
+@register_stream_part("add_turn_vector")
+class TurnVector(StreamPart):
+    """params: ``hidden_size``, ``turns`` (runs of the stretch).  Tensor ``weight`` [turns, hidden]."""
+
+    wants_turn = True
+
+    def __init__(self, spec, dtype, device):
+        super().__init__(spec, dtype, device)
+        self.hidden = int(spec["hidden_size"])
+        self.turns = int(spec["turns"])
+        self.rows = None
+
+    def tensors(self) -> Dict[str, TensorSpec]:
+        return {"weight": TensorSpec((self.turns, self.hidden))}
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        table = tensors["weight"].to(torch.float32)
+        self.rows = [table[t].clone() for t in range(self.turns)]       # tensors of their own: 16-byte aligned whatever the width
+
+    def kernel_libraries(self):
+        return ("tanh_norm",)
+
+    def forward(self, residual: torch.Tensor, delta, ctx, turn: int = 0):
+        row = self.rows[turn]
+        if isinstance(delta, TanhAddend) and delta.row is None:
+            return residual, TanhAddend(delta.y, delta.alpha, delta.weight, delta.bias, row)
+        ops.kernels().add_row(residual, row)
+        return residual, delta

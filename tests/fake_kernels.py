@@ -559,8 +559,91 @@ class FakeKernels:
             rows = rows * weights.view(n, top, 1)
         out.copy_((rows.sum(1) + add.float()).to(out.dtype))
 
+    # ---- a norm by tanh -------------------------------------------------------------------------------------------------
+    def tanh_add_tanh(self, residual, y, alpha_y, weight_y, bias_y, row, alpha, weight, bias, out):
+        if y is not None:
+            v = y.float()
+            residual.add_(torch.tanh(alpha_y * v) * weight_y + bias_y if weight_y is not None else v)
+        if row is not None:
+            residual.add_(row)
+        if out is not None:
+            out.copy_((torch.tanh(alpha * residual) * weight + bias).to(out.dtype))
+
+    def add_row(self, residual, row):
+        residual.add_(row)
+
+    # ---- heads as the difference of two softmax maps ------------------------------------------------------------------------
+    def rotate_pairs_store(self, proj, q_off, k_off, v_off, q_out, k_cache, v_cache, table, slots, *, num_heads, num_kv_heads, maps,
+                           k_dim, v_dim, rot_dim):
+        n = proj.shape[0]
+
+        def turn(cols, heads):
+            t = cols.reshape(n, heads, k_dim).float().clone()
+            if rot_dim:
+                cos, sin = table[:, None, :, 0], table[:, None, :, 1]
+                a, b = t[..., 0:rot_dim:2].clone(), t[..., 1:rot_dim:2].clone()
+                t[..., 0:rot_dim:2] = a * cos - b * sin
+                t[..., 1:rot_dim:2] = b * cos + a * sin
+            return t
+
+        q_out.copy_(turn(proj[:, q_off:q_off + num_heads * k_dim], num_heads).reshape(n, -1).to(q_out.dtype))
+        if k_cache is None:
+            return
+        k = turn(proj[:, k_off:k_off + num_kv_heads * maps * k_dim], num_kv_heads * maps).reshape(n, num_kv_heads, maps * k_dim)
+        v = proj[:, v_off:v_off + num_kv_heads * v_dim].reshape(n, num_kv_heads, v_dim)
+        ps = k_cache.shape[2]
+        for t in range(n):
+            c = int(slots[t])
+            if c >= 0:
+                k_cache[c // ps, :, c % ps, :] = k[t].to(k_cache.dtype)
+                v_cache[c // ps, :, c % ps, :] = v[t].to(v_cache.dtype)
+
+    def difference_attention(self, q, k_cache, v_cache, out, meta, *, num_heads, num_kv_heads, k_dim, v_dim, scale, softcap, lam,
+                             factor, eps, **_):
+        n = q.shape[0]
+        ps = k_cache.shape[2]
+        rep = num_heads // num_kv_heads
+        qf = q.float().reshape(n, num_heads, 2, k_dim)
+        o = torch.zeros(n, num_heads, v_dim)
+        for t in range(n):
+            s = int(meta.seq_of_token[t])
+            if s < 0:
+                continue
+            js = torch.arange(int(meta.positions[t]) + 1)
+            pages = meta.block_table[s, (js // ps).long()].long()
+            assert (pages >= 0).all(), "attention reads a page that was given back"
+            kk = k_cache[pages, :, (js % ps).long(), :].float().view(js.numel(), num_kv_heads, 2, k_dim)
+            vv = v_cache[pages, :, (js % ps).long(), :].float()
+            for h in range(num_heads):
+                sc = torch.einsum("jmd,md->mj", kk[:, h // rep], qf[t, h]) * scale
+                if softcap:
+                    sc = softcap * torch.tanh(sc / softcap)
+                a = torch.softmax(sc, dim=-1) @ vv[:, h // rep, :]
+                d = a[0] - lam * a[1]
+                o[t, h] = d / torch.sqrt((d * d).mean() + eps) * factor
+        out.copy_(o.view(n, num_heads * v_dim).to(out.dtype))
+
+    def relu2(self, x, out):
+        out.copy_((torch.relu(x.float()) ** 2).to(out.dtype))
+
+    def moe_route_corrected(self, logits, correction, top, ids, weights, scale):
+        s = torch.softmax(logits.float(), dim=-1)
+        order = torch.sort(s + (correction if correction is not None else 0.0), dim=-1, descending=True, stable=True).indices[:, :top]
+        ids.copy_(order.int())
+        weights.copy_(scale * torch.gather(s, 1, order))
+
+    def moe_combine_mixed(self, ys, pos, weights, h, out, top, add, add_gate):
+        n = out.shape[0]
+        rows = ys[pos.long().clamp(min=0)].float().view(n, top, -1)
+        own = (pos.view(n, top, 1) < 0)
+        y = (torch.where(own, h.float()[:, None, :], rows) * weights.view(n, top, 1)).sum(1)
+        if add is not None:
+            y = y + (torch.sigmoid(add_gate) if add_gate is not None else 1.0) * add.float()
+        out.copy_(y.to(out.dtype))
+
     # ---- the delta rule with a decay per key channel --------------------------------------------------------
-    def delta_rule(self, proj, col_off, b_off, z, taps, a_log, dt_bias, state, ctx, out, *, num_heads, num_kv_heads, dim, v_dim):
+    def delta_rule(self, proj, col_off, b_off, z, taps, a_log, dt_bias, state, ctx, out, *, num_heads, num_kv_heads, dim, v_dim,
+                   b_pre=None):
         H, G, D, V = num_heads, num_kv_heads, dim, v_dim
         C = 2 * G * D + H * V
         n_taps = taps.shape[1]
@@ -587,8 +670,8 @@ class FakeKernels:
                 k = k / torch.sqrt((k * k).sum(-1, keepdim=True) + 1e-6)
                 q, k = q.repeat_interleave(H // G, dim=0), k.repeat_interleave(H // G, dim=0)
                 v = a[2 * G * D:].view(H, V)
-                beta = torch.sigmoid(proj[t, b_off:b_off + H].float())
-                g = torch.exp(-torch.exp(a_log)[:, None] * sp(z[t].view(H, D) + dt_bias.view(H, D)))
+                beta = torch.sigmoid(b_pre[t] if b_pre is not None else proj[t, b_off:b_off + H].float())
+                g = torch.exp(-torch.exp(a_log)[:, None] * sp(z[t].reshape(H, -1) + dt_bias.view(H, -1)))      # [H, D] or [H, 1]
                 S = S * g[:, None, :]
                 u = beta[:, None] * (v - torch.einsum("hvd,hd->hv", S, k))
                 S = S + u[:, :, None] * k[:, None, :]
@@ -611,15 +694,19 @@ class FakeKernels:
 
     def moe_plan(self, ids, num_experts, offsets, pos, tiles, tile_rows=None):
         flat = ids.reshape(-1).long()
+        flat = torch.where(flat < num_experts, flat, torch.full_like(flat, num_experts))     # no expert behind it: no row
         order = torch.sort(flat, stable=True).indices
         pos[order] = torch.arange(flat.numel(), dtype=pos.dtype)
-        counts = torch.bincount(flat, minlength=num_experts)
+        pos[flat == num_experts] = -1
+        counts = torch.bincount(flat, minlength=num_experts + 1)[:num_experts]
         offsets[0] = 0
         offsets[1:] = torch.cumsum(counts, 0).int()
 
     def moe_scatter(self, h, pos, weights, xs, top):
         w = weights.reshape(-1) if weights is not None else torch.ones(pos.numel())
         for i in range(pos.numel()):
+            if int(pos[i]) < 0:
+                continue
             xs[int(pos[i])] = (w[i] * h[i // top].float()).to(xs.dtype)
 
     def moe_grouped_gemm(self, x, w, w2, out, offsets, tiles, activation="silu", limit=0.0):
@@ -638,6 +725,8 @@ class FakeKernels:
                     y = g * torch.sigmoid(1.702 * g) * (u + 1.0)
                 else:
                     y = self._act(g, activation) * u
+            elif activation == "relu2":
+                y = torch.relu(y) ** 2
             out[a:b] = y.to(out.dtype)
 
     def moe_combine(self, ys, pos, out, top, weights=None):
