@@ -24,6 +24,13 @@
 // position p iff j <= p and (window == 0 or p - j < window); softmax in float32; o = sum p_j v_j; a row that
 // sees no key yields zeros.
 //
+// The difference form (heads that are the difference of two softmax maps over the same values; see difference_attention.cu): a key
+// cell's halves are the two maps' keys and a query row's halves the two maps' queries, so a CTA owns 128 rows and its groups are
+// the MAPS: group m multiplies the half tiles m of Q and K, and both multiply their P with the same V.  Scores pass a tanh cap
+// before the softmax: as an odd polynomial of the score in packed float32 pairs where every |score| of a warp's rows in the tile
+// is within half the cap, else by the exponential and reciprocal units.  At the end the groups' outputs, which lie in the
+// same lanes of tensor memory, are subtracted, each group taking one half of the columns.
+//
 // Every wait on an mbarrier is bounded: after kSpinLimit polls the waiter records where it gave up in
 // `status`, and every role falls through to the common exit, where tensor memory is freed.
 #include <cuda.h>
@@ -66,6 +73,11 @@ struct TcAttnParams {
     int keep_first = 0;
     // one gate number per head (rows of nh numbers) instead of one per entry
     int gate_per_head = 0;
+    // difference form: t = cap_out * tanh(cap_in * s) takes the place of s (then scale_log2 is 1); cap_in 0: no cap
+    float cap_in = 0.0f, cap_out = 0.0f;
+    float cap_poly[4] = {0.0f, 0.0f, 0.0f, 0.0f};   // t = s (c0 + c1 s^2 + c2 s^4 + c3 s^6) for |s| <= cap_small
+    float cap_small = 0.0f;
+    float lambda = 0.0f, factor = 0.0f, eps = 0.0f;
 };
 
 __device__ __forceinline__ unsigned at_smem(const void * p) { return (unsigned) __cvta_generic_to_shared(p); }
@@ -144,6 +156,22 @@ __device__ __forceinline__ unsigned long long at_fma2(unsigned long long a, unsi
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
     return r;
 }
+__device__ __forceinline__ unsigned long long at_mul2(unsigned long long a, unsigned long long b) {
+    unsigned long long r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ float at_min3(float a, float b, float c) {
+    float r;
+    asm("min.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c));
+    return r;
+}
+__device__ __forceinline__ float at_tanh(float x) {      // 1 - 2 / (1 + e^2x), absolute error of a few 1e-7
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+    return fmaf(-2.0f, r, 1.0f);
+}
 __device__ __forceinline__ unsigned long long at_add2(unsigned long long a, unsigned long long b) {
     unsigned long long r;
     asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
@@ -178,10 +206,14 @@ __host__ __device__ constexpr unsigned at_idesc(int m, int n, bool b_mn) {
     return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn ? (1u << 16) : 0u) | ((unsigned) (n >> 3) << 17) | ((unsigned) (m >> 4) << 24);
 }
 
-// KEPT: the form with kept first keys and a gate per head is an instance of its own, so that the other stays as it was
-template <bool KEPT>
+// The form with kept first keys and a gate per head (AT_KEPT) and the difference form (AT_DIFF) are instances of their own, so that
+// the plain one stays as it was
+enum { AT_PLAIN = 0, AT_KEPT = 1, AT_DIFF = 2 };
+template <int FORM>
 __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
     const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const TcAttnParams p) {
+    constexpr bool KEPT = FORM == AT_KEPT, DIFF = FORM == AT_DIFF;
+    constexpr int CTA_ROWS = DIFF ? AT_BM : AT_ROWS;
     extern __shared__ __align__(1024) unsigned char at_smem_raw[];
     unsigned char * smem = (unsigned char *) (((uintptr_t) at_smem_raw + 1023) & ~(uintptr_t) 1023);
     unsigned char * sQ = smem;                               // [2 groups][2 halves][128 rows][128 B]
@@ -198,14 +230,14 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
     const int ctx = p.ctx_len[s];
     const int pos0 = ctx - q_len;
     const int rows_total = q_len * G;
-    const int row0 = ((int) gridDim.x - 1 - (int) blockIdx.x) * AT_ROWS;    // late rows see the most keys: they start first
+    const int row0 = ((int) gridDim.x - 1 - (int) blockIdx.x) * CTA_ROWS;    // late rows see the most keys: they start first
     if (row0 >= rows_total) return;
 
     // two groups of 128 rows (A, B) share every K/V tile; B may be empty, and A may need a tile less than B
-    const bool has_b = row0 + AT_BM < rows_total;
+    const bool has_b = DIFF || row0 + AT_BM < rows_total;
     const int tok_min = row0 / G;
     const int k_hi_a = pos0 + min(rows_total - 1, row0 + AT_BM - 1) / G;
-    const int k_hi = pos0 + min(rows_total - 1, row0 + AT_ROWS - 1) / G;
+    const int k_hi = pos0 + min(rows_total - 1, row0 + CTA_ROWS - 1) / G;
     const int k_lo = p.window > 0 ? max(0, pos0 + tok_min - p.window + 1)
                                   : p.chunk > 0 ? (pos0 + tok_min) - (pos0 + tok_min) % p.chunk : 0;
     const int tile_lo = k_lo / AT_BN, tile_hi = k_hi / AT_BN;
@@ -249,7 +281,7 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
         // loads of a pass are all issued before the first is stored, so that a pass costs one trip to memory.
         constexpr int kLoaders = AT_THREADS - 32, kPass = 8;
         const int t = threadIdx.x - 32;
-        for (int base = 0; base < AT_ROWS * 16; base += kLoaders * kPass) {
+        for (int base = 0; base < CTA_ROWS * 16; base += kLoaders * kPass) {
             uint4 buf[kPass];
 #pragma unroll
             for (int u = 0; u < kPass; u++) {
@@ -257,7 +289,7 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
                 const int rr = idx >> 4, c = idx & 15;
                 const int R = row0 + rr;
                 buf[u] = make_uint4(0u, 0u, 0u, 0u);
-                if (idx < AT_ROWS * 16 && R < rows_total) {
+                if (idx < CTA_ROWS * 16 && R < rows_total) {
                     const int tok = R / G, head = kvh * G + R % G;
                     buf[u] = *reinterpret_cast<const uint4 *>(p.q + (size_t) (q0 + tok) * p.ld_q + (size_t) head * AT_HD + c * 8);
                 }
@@ -265,10 +297,13 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
 #pragma unroll
             for (int u = 0; u < kPass; u++) {
                 const int idx = base + u * kLoaders + t;
-                if (idx < AT_ROWS * 16) {
+                if (idx < CTA_ROWS * 16) {
                     const int rr = idx >> 4, c = idx & 15;
-                    const int g = rr >> 7, r = rr & 127;
-                    *reinterpret_cast<uint4 *>(sQ + g * AT_TILE_BYTES + (c >> 3) * AT_HALF_BYTES + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = buf[u];
+                    const int g = DIFF ? c >> 3 : rr >> 7, r = rr & 127;
+                    if constexpr (DIFF)               // a row's halves are the maps: each group's tile is one half tile
+                        *reinterpret_cast<uint4 *>(sQ + g * AT_TILE_BYTES + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = buf[u];
+                    else
+                        *reinterpret_cast<uint4 *>(sQ + g * AT_TILE_BYTES + (c >> 3) * AT_HALF_BYTES + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = buf[u];
                 }
             }
         }
@@ -341,10 +376,17 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
         // P V of the tile before in program order (the tensor pipe runs a thread's MMAs in order).
         auto issue_qk = [&](int g, int i) {
             const int st = i & 1;
+            if constexpr (DIFF) {
 #pragma unroll
-            for (int k = 0; k < 8; k++) {             // 16 values of the head per step: 32 bytes inside the atom, halves 16 KB apart
-                const unsigned long long off = (unsigned long long) ((k >> 2) * kHalf16 + (k & 3) * 2);
-                at_mma(tmem_base + (unsigned) (g * 128), dq[g] + off, dk[st] + off, idesc_qk, k > 0 ? 1u : 0u);
+                for (int k = 0; k < 4; k++)           // the map's 64 values: half tile g of K
+                    at_mma(tmem_base + (unsigned) (g * 128), dq[g] + (unsigned long long) (k * 2), dk[st] + (unsigned long long) (g * kHalf16 + k * 2),
+                           idesc_qk, k > 0 ? 1u : 0u);
+            } else {
+#pragma unroll
+                for (int k = 0; k < 8; k++) {         // 16 values of the head per step: 32 bytes inside the atom, halves 16 KB apart
+                    const unsigned long long off = (unsigned long long) ((k >> 2) * kHalf16 + (k & 3) * 2);
+                    at_mma(tmem_base + (unsigned) (g * 128), dq[g] + off, dk[st] + off, idesc_qk, k > 0 ? 1u : 0u);
+                }
             }
             at_commit(at_smem(&s_full[g]));
         };
@@ -378,7 +420,7 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
         const int g = (warp - 2) >> 2;
         const int qd = warp & 3;
         const int r = qd * 32 + lane;
-        const int R = row0 + g * AT_BM + r;
+        const int R = row0 + (DIFF ? 0 : g * AT_BM) + r;
         const bool row_ok = R < rows_total;
         const int row_pos = pos0 + (row_ok ? R / G : 0);
         const unsigned lane_addr = (unsigned) (qd * 32) << 16;
@@ -408,6 +450,36 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
 #pragma unroll
             for (int c0 = 0; c0 < AT_BN; c0 += 32) at_ld32(tS + lane_addr + (unsigned) c0, v + c0);
             at_wait_ld();
+            if constexpr (DIFF) {
+                if (p.cap_in > 0.0f) {                // t = cap_out tanh(cap_in s), of every column (hidden ones are set below)
+                    float hi4[2] = {0.0f, 0.0f}, lo4[2] = {0.0f, 0.0f};
+#pragma unroll
+                    for (int j = 0; j < AT_BN; j += 4) {
+                        hi4[0] = at_max3(hi4[0], __uint_as_float(v[j]), __uint_as_float(v[j + 1]));
+                        lo4[0] = at_min3(lo4[0], __uint_as_float(v[j]), __uint_as_float(v[j + 1]));
+                        hi4[1] = at_max3(hi4[1], __uint_as_float(v[j + 2]), __uint_as_float(v[j + 3]));
+                        lo4[1] = at_min3(lo4[1], __uint_as_float(v[j + 2]), __uint_as_float(v[j + 3]));
+                    }
+                    const float far = fmaxf(fmaxf(hi4[0], hi4[1]), -fminf(lo4[0], lo4[1]));
+                    if (__all_sync(0xffffffffu, far <= p.cap_small)) {
+                        const unsigned long long c0 = at_pack2(p.cap_poly[0], p.cap_poly[0]), c1 = at_pack2(p.cap_poly[1], p.cap_poly[1]);
+                        const unsigned long long c2 = at_pack2(p.cap_poly[2], p.cap_poly[2]), c3 = at_pack2(p.cap_poly[3], p.cap_poly[3]);
+#pragma unroll
+                        for (int j = 0; j < AT_BN; j += 2) {
+                            const unsigned long long x = at_pack2(__uint_as_float(v[j]), __uint_as_float(v[j + 1]));
+                            const unsigned long long x2 = at_mul2(x, x);
+                            const unsigned long long y = at_mul2(x, at_fma2(x2, at_fma2(x2, at_fma2(x2, c3, c2), c1), c0));
+                            float y0, y1;
+                            at_unpack2(y, y0, y1);
+                            v[j] = __float_as_uint(y0);
+                            v[j + 1] = __float_as_uint(y1);
+                        }
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < AT_BN; j++) v[j] = __float_as_uint(p.cap_out * at_tanh(p.cap_in * __uint_as_float(v[j])));
+                    }
+                }
+            }
             // visible keys of this row in this tile: columns [lo, hi]; most tiles lie wholly below the diagonal
             const int hi = row_ok ? min(AT_BN - 1, row_pos - key0) : -1;
             int lo = p.window > 0 ? max(0, row_pos - p.window + 1 - key0) : max(0, row_lo - key0);
@@ -496,6 +568,51 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
             __syncwarp();
             if (lane == 0) at_arrive(at_smem(&p_full[g]));
         }
+        if constexpr (DIFF) {
+            // ---- map 1 - lambda * map 2, over the root mean square -> out: both maps' outputs of a row lie in the same lane; a
+            // group's thread takes 64 of the row's columns
+            __shared__ float x_l[2][AT_BM], x_ss[2][AT_BM];
+            x_l[g][r] = l_run;
+            // each group waits for its OWN last product (it has followed that barrier phase by phase); the barrier then tells the other
+            const bool good = !failed && at_wait(at_smem(&pv_done[g]), (unsigned) (n_mine - 1) & 1u);
+            if (!good && lane == 0) { status[0] = 9; status[1] = n_mine; }
+            at_fence_after();
+            at_fence_before();
+            asm volatile("bar.sync 1, 256;" ::: "memory");           // the eight softmax warps
+            at_fence_after();
+            const float l0 = x_l[0][r], l1 = x_l[1][r];
+            const float i0 = l0 > 0.0f ? 1.0f / l0 : 0.0f, i1 = l1 > 0.0f ? p.lambda / l1 : 0.0f;
+            const unsigned t0 = tmem_base + 256u + lane_addr + (unsigned) (g * 64);
+            float o[64], ss = 0.0f;
+#pragma unroll
+            for (int c0 = 0; c0 < 64; c0 += 32) {
+                unsigned a[32], b[32];
+                at_ld32(t0 + (unsigned) c0, a);
+                at_ld32(t0 + 128u + (unsigned) c0, b);
+                at_wait_ld();
+#pragma unroll
+                for (int j = 0; j < 32; j++) {
+                    o[c0 + j] = __uint_as_float(a[j]) * i0 - __uint_as_float(b[j]) * i1;
+                    ss = fmaf(o[c0 + j], o[c0 + j], ss);
+                }
+            }
+            x_ss[g][r] = ss;
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            if (row_ok && good) {
+                const float f = p.factor / sqrtf((x_ss[0][r] + x_ss[1][r]) / (float) AT_HD + p.eps);
+                const int tok = R / G, head = kvh * G + R % G;
+                __nv_bfloat16 * dst = p.out + ((size_t) (q0 + tok) * p.nh + head) * AT_HD + g * 64;
+#pragma unroll
+                for (int q8 = 0; q8 < 8; q8++) {
+                    uint4 pk;
+                    __nv_bfloat162 h0 = __floats2bfloat162_rn(o[8 * q8 + 0] * f, o[8 * q8 + 1] * f), h1 = __floats2bfloat162_rn(o[8 * q8 + 2] * f, o[8 * q8 + 3] * f);
+                    __nv_bfloat162 h2 = __floats2bfloat162_rn(o[8 * q8 + 4] * f, o[8 * q8 + 5] * f), h3 = __floats2bfloat162_rn(o[8 * q8 + 6] * f, o[8 * q8 + 7] * f);
+                    pk.x = *reinterpret_cast<unsigned *>(&h0); pk.y = *reinterpret_cast<unsigned *>(&h1);
+                    pk.z = *reinterpret_cast<unsigned *>(&h2); pk.w = *reinterpret_cast<unsigned *>(&h3);
+                    *reinterpret_cast<uint4 *>(dst + 8 * q8) = pk;
+                }
+            }
+        } else
         // ---- O / sum -> out ---------------------------------------------------------------------------
         if (n_mine > 0 && !failed) {
             if (at_wait(at_smem(&pv_done[g]), (unsigned) (n_mine - 1) & 1u)) {
@@ -681,14 +798,60 @@ IIAN_API int iian_attention_tc_kept(const void * q, long long ld_q, const void *
     const bool kept = keep_first > 0 || p.gate_per_head;
     static bool configured[2] = {false, false};
     if (!configured[kept ? 1 : 0]) {
-        cudaError_t e = kept ? cudaFuncSetAttribute(attention_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem)
-                             : cudaFuncSetAttribute(attention_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
+        cudaError_t e = kept ? cudaFuncSetAttribute(attention_tc_kernel<AT_KEPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem)
+                             : cudaFuncSetAttribute(attention_tc_kernel<AT_PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
         if (e != cudaSuccess) return 1000 + (int) e;
         configured[kept ? 1 : 0] = true;
     }
     const int max_rows = max_q_len * (nh / nkv);
     dim3 grid((max_rows + AT_ROWS - 1) / AT_ROWS, nkv, S);
-    if (kept) attention_tc_kernel<true><<<grid, AT_THREADS, smem, stream>>>(mk, mv, p);
-    else attention_tc_kernel<false><<<grid, AT_THREADS, smem, stream>>>(mk, mv, p);
+    if (kept) attention_tc_kernel<AT_KEPT><<<grid, AT_THREADS, smem, stream>>>(mk, mv, p);
+    else attention_tc_kernel<AT_PLAIN><<<grid, AT_THREADS, smem, stream>>>(mk, mv, p);
+    return iian_launch_status();
+}
+
+// The difference form: q [N, nh, 2, 64], caches [num_pages, nkv, page_size, 128] (a key cell holds both maps' keys), out
+// [N, nh * 128].  Per map scores q . k * scale, then cap * tanh(./cap) (cap 0: as they are), causal, softmax; out = (map 1 - lambda
+// * map 2) / root mean square * factor.  scale > 0; page sizes and status as for the other forms.
+IIAN_API int iian_attention_tc_difference(const void * q, const void * k_cache, const void * v_cache, void * out, const int * cu_q,
+                                          const int * ctx_len, const int * block_table, int max_blocks, int N, int S, int max_q_len,
+                                          int nh, int nkv, int page_size, int num_pages, float scale, float cap, float lambda,
+                                          float factor, float eps, int * status, cudaStream_t stream) {
+    if (N <= 0 || S <= 0) return IIAN_OK;
+    if (nkv <= 0 || nh % nkv != 0 || !(scale > 0.0f) || cap < 0.0f || status == nullptr) return IIAN_ERR_SHAPE;
+    if (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64 && page_size != 128) return IIAN_ERR_SHAPE;
+    if (((uintptr_t) q & 15) || ((uintptr_t) k_cache & 15) || ((uintptr_t) v_cache & 15) || ((uintptr_t) out & 15)) return IIAN_ERR_ALIGN;
+    if (S > 65535 || nkv > 65535) return IIAN_ERR_LIMIT;
+    CUtensorMap mk, mv;
+    int rc = at_make_map(&mk, k_cache, num_pages, nkv, page_size);
+    if (rc != IIAN_OK) return rc;
+    rc = at_make_map(&mv, v_cache, num_pages, nkv, page_size);
+    if (rc != IIAN_OK) return rc;
+    TcAttnParams p;
+    p.q = (const __nv_bfloat16 *) q; p.out = (__nv_bfloat16 *) out; p.cu_q = cu_q; p.ctx_len = ctx_len; p.block_table = block_table;
+    p.max_blocks = max_blocks; p.nh = nh; p.nkv = nkv; p.page_size = page_size; p.num_pages = num_pages; p.window = 0;
+    p.scale_log2 = cap > 0.0f ? 1.0f : scale * 1.4426950408889634f;
+    p.status = status;
+    p.ld_q = (long long) nh * AT_HD;
+    p.lambda = lambda; p.factor = factor; p.eps = eps;
+    if (cap > 0.0f) {
+        // tanh(x) = x (a0 + a1 x^2 + a2 x^4 + a3 x^6) for |x| <= 1/2, fitted for the least largest error (1.3e-7 absolute)
+        static const double a[4] = {0.999997675672, -0.333206535381, 0.131451321517, -0.0433721740216};
+        const double c = (double) scale / cap, out_scale = (double) cap * 1.4426950408889634;
+        p.cap_in = (float) c;
+        p.cap_out = (float) out_scale;
+        double f = out_scale * c;
+        for (int i = 0; i < 4; i++, f *= c * c) p.cap_poly[i] = (float) (f * a[i]);
+        p.cap_small = (float) (0.5 / c);
+    }
+    const size_t smem = (size_t) 6 * AT_TILE_BYTES + 1024;
+    static bool configured = false;
+    if (!configured) {
+        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<AT_DIFF>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
+        if (e != cudaSuccess) return 1000 + (int) e;
+        configured = true;
+    }
+    dim3 grid((max_q_len * (nh / nkv) + AT_BM - 1) / AT_BM, nkv, S);
+    attention_tc_kernel<AT_DIFF><<<grid, AT_THREADS, smem, stream>>>(mk, mv, p);
     return iian_launch_status();
 }

@@ -27,12 +27,14 @@ ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 BASE_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--shared", "-Xcompiler", "-fPIC,-fvisibility=hidden",
               "--expt-relaxed-constexpr"]
 SHARED_HEADERS = ["common.cuh"]
+# further headers that some sources share
+SOURCE_HEADERS: Dict[str, List[str]] = {"attention_mma": ["paged_mma.cuh"], "difference_attention_mma": ["paged_mma.cuh"]}
 
 # every library of the engine; build_all() compiles them all
 SOURCES = ["elementwise", "rope_kv", "attention_generic", "gemm_simt", "sampling", "gemm_skinny", "attention_mma", "prefetch", "gemm_tcgen05",
            "attention_tc", "gemm_stream", "postnorm", "latent_attention", "moe", "latent_attention_mma",
            "stream_ops", "shared_kv", "matrix_memory", "residual_ops", "chunked_attention", "delta_rule", "window_attention",
-           "decay_scan", "tanh_norm", "difference_attention"]
+           "decay_scan", "tanh_norm", "difference_attention", "difference_attention_mma"]
 # libraries only the bfloat16 serving path uses
 BF16_SOURCES: List[str] = ["gemm_skinny", "attention_mma", "prefetch", "gemm_tcgen05", "attention_tc", "gemm_stream"]
 BF16_PRODUCT_SOURCES: List[str] = ["gemm_skinny", "gemm_tcgen05", "gemm_stream"]
@@ -90,7 +92,7 @@ def _pick_build_dir() -> str:
 
 def _source_hash(name: str) -> str:
     h = hashlib.sha256()
-    for fn in [f"{name}.cu"] + SHARED_HEADERS:
+    for fn in [f"{name}.cu"] + SHARED_HEADERS + SOURCE_HEADERS.get(name, []):
         p = os.path.join(HERE, fn)
         if os.path.isfile(p):
             with open(p, "rb") as f:

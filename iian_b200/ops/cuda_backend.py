@@ -1713,18 +1713,59 @@ class CudaKernels:
                   _cuda(table if rot_dim else None, "rotary table"), _cuda(slots, "slots", torch.int32), _code(proj, "projections"), n,
                   num_heads, num_kv_heads, maps, k_dim, v_dim, rot_dim, page, cells, _stream()), "rotate_pairs_store")
 
+    # tensor-core forms; IIAN_DIFFERENCE_ATTENTION_MMA=0: the general kernel in bfloat16 too
+    DIFFERENCE_ATTENTION_MMA = os.environ.get("IIAN_DIFFERENCE_ATTENTION_MMA", "1") not in ("0", "false", "off")
+
+    def difference_attention_mma_ok(self, dtype, k_dim: int, v_dim: int, scale: float) -> bool:
+        return self.DIFFERENCE_ATTENTION_MMA and dtype == torch.bfloat16 and k_dim == 64 and v_dim == 128 and scale > 0
+
+    def difference_splits(self, num_seqs: int, num_kv_heads: int, max_ctx: int) -> int:
+        """Parts of the keys of a decode step: as for plain heads, but never more than a cluster holds."""
+        return min(16, self.attention_splits(num_seqs, num_kv_heads, max_ctx))
+
+    def difference_attention_plan(self, num_seqs: int, num_kv_heads: int, k_dim: int, v_dim: int, scale: float, max_ctx: int, dtype):
+        if not self.difference_attention_mma_ok(dtype, k_dim, v_dim, scale):
+            return None
+        return {"n_split": self.difference_splits(num_seqs, num_kv_heads, max_ctx)}
+
     def difference_attention(self, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, meta, *,
                              num_heads: int, num_kv_heads: int, k_dim: int, v_dim: int, scale: float, softcap: Optional[float],
-                             lam: float, factor: float, eps: float) -> None:
+                             lam: float, factor: float, eps: float, n_split: Optional[int] = None) -> None:
         """``q`` [N, heads * 2 * k_dim] -> ``out`` [N, heads * v_dim]: per head the two maps' softmax (scores ``q . k * scale``,
         then ``softcap tanh(./softcap)``; causal) over the cached keys, ``o = a1 - lam a2`` of the values both share, ``o``
-        divided by its root mean square over the head, times ``factor``."""
+        divided by its root mean square over the head, times ``factor``.  In bfloat16 with maps of 64 and values of 128 the
+        tensor-core kernels serve it: long portions ``csrc/attention_tc.cu``, decoded tokens and short portions
+        ``csrc/difference_attention_mma.cu`` (``n_split`` parts of the keys); otherwise the general kernel of
+        ``csrc/difference_attention.cu``."""
         n = q.shape[0]
         if q.shape[1] != num_heads * 2 * k_dim or out.shape != (n, num_heads * v_dim) or out.dtype != q.dtype \
                 or k_cache.dtype != q.dtype or k_cache.shape[3] != 2 * k_dim or v_cache.shape[3] != v_dim \
                 or k_cache.shape[1] != num_kv_heads:
             raise KernelError(f"difference_attention: q {tuple(q.shape)}, out {tuple(out.shape)}, cache {tuple(k_cache.shape)} do not fit")
         bt = meta.block_table
+        if self.difference_attention_mma_ok(q.dtype, k_dim, v_dim, scale) and n:
+            group = num_heads // num_kv_heads
+            page = k_cache.shape[2]
+            status = self.tcgen05_status_buffer(q.device)
+            CudaKernels._tc_used = True
+            common = [_cuda(q, "queries"), _cuda(k_cache, "key cache"), _cuda(v_cache, "value cache"), _cuda(out, "attention out"),
+                      _cuda(meta.cu_q, "cu_q", torch.int32), _cuda(meta.ctx_len, "ctx_len", torch.int32),
+                      _cuda(bt, "block table", torch.int32), bt.shape[1]]
+            if self.ATTENTION_TC and page in (8, 16, 32, 64, 128) and meta.max_q_len * group >= self.TC_ATTENTION_MIN_ROWS:
+                fn = _fn("attention_tc", "iian_attention_tc_difference",
+                         [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                          c_int, c_int, c_float, c_float, c_float, c_float, c_float, c_void_p, c_void_p])
+                _check(fn(*common, n, meta.num_seqs, meta.max_q_len, num_heads, num_kv_heads, page, k_cache.shape[0], scale,
+                          softcap or 0.0, lam, factor, eps, status.data_ptr(), _stream()), "attention_tc_difference")
+                return
+            if n_split is None:
+                n_split = self.difference_splits(meta.num_seqs, num_kv_heads, meta.max_ctx) if meta.max_q_len * group <= 16 else 1
+            fn = _fn("difference_attention_mma", "iian_difference_attention_mma",
+                     [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                      c_float, c_float, c_float, c_float, c_float, c_int, c_void_p, c_void_p])
+            _check(fn(*common, meta.num_seqs, meta.max_q_len, num_heads, num_kv_heads, page, k_cache.shape[0], scale, softcap or 0.0, lam,
+                      factor, eps, n_split, self._decode_status(q.device), _stream()), "difference_attention_mma")
+            return
         fn = _fn("difference_attention", "iian_difference_attention",
                  [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
                   c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_float, c_void_p])

@@ -89,10 +89,17 @@ class DifferenceAttention(Mixer):
         return KVNeed(self.nkv, 2 * self.hd, None, self.vd if self.vd != 2 * self.hd else None)
 
     def _fast(self) -> bool:
-        return self.dtype == torch.bfloat16 and self.hd == 64 and self.vd == 128
+        return self.dtype == torch.bfloat16 and self.hd == 64 and self.vd == 128 and self.scale > 0
 
     def kernel_libraries(self):
-        return ("difference_attention", "gemm_simt") + (("window_attention",) if self.rot else ())
+        return ("difference_attention", "gemm_simt") + (("window_attention",) if self.rot else ()) \
+            + (("difference_attention_mma", "attention_tc") if self._fast() else ())
+
+    def graph_plan(self, num_seqs: int, max_ctx: int):
+        k = ops.kernels()
+        if not hasattr(k, "difference_attention_plan"):
+            return None
+        return k.difference_attention_plan(num_seqs, self.nkv, self.hd, self.vd, self.scale, max_ctx, self.dtype)
 
     def forward(self, x, ctx, cache, writes_cache: bool):
         if not writes_cache:
@@ -106,10 +113,11 @@ class DifferenceAttention(Mixer):
         q = ctx.buf("q", (n, self.q_size), self.dtype)
         k.rotate_pairs_store(proj, 0, self.q_size, self.q_size + self.k_size, q, cache.k, cache.v, table, meta.slots,
                              num_heads=2 * self.nh, num_kv_heads=self.nkv, maps=2, k_dim=self.hd, v_dim=self.vd, rot_dim=self.rot)
+        plan = ctx.graph_plan(self)
         attn = ctx.buf("attn", (n, self.nh * self.vd), self.dtype)
         k.difference_attention(q, cache.k, cache.v, attn, meta, num_heads=self.nh, num_kv_heads=self.nkv, k_dim=self.hd,
                                v_dim=self.vd, scale=self.scale, softcap=self.softcap, lam=self.lam, factor=1.0 - self.diff,
-                               eps=self.eps)
+                               eps=self.eps, **({"n_split": plan["n_split"]} if plan else {}))
         out = ctx.buf("mixer_out", (n, self.hidden), self.dtype)
         k.linear(attn, self.w_o, out)
         return out
