@@ -583,6 +583,162 @@ def run_nogelorn(peaks: dict, width: int = 2048, heads: int = 16) -> dict:
     return out
 
 
+def run_ferodra(peaks: dict, width: int = 2048, heads: int = 16) -> dict:
+    """The kernels of the Ferodra design alone, each beside its like kernel at equal size (16 heads whose two maps are 64 wide over
+    values of 128, on 8 KV heads):
+      decode attention    8 (and 64) sequences of 4,096 cached tokens  vs  Qwen3's plain heads of 128 (the same bytes of cache)
+      prefill attention   one sequence of 2,048 tokens, and of 8,192  vs  Qwen3's
+      rotation + cache    2,048 tokens  vs  Nogelorn's rotation, unit norm, cache write
+      sum + norm          2,048 rows: an addend normalised by tanh in the next norm by tanh  vs  Nogelorn's RMS forms
+      expert products     2,048 (and 8) tokens x 5 of 64 ungated experts and 4 identity outputs + a gated shared one  vs  Nogelorn's
+                          5 of 64 gated ones of equal weights + a shared one
+      delta rule          8 / 64 sequences of one token (bytes of state) and one sequence of 2,048 tokens, one decay per head  vs
+                          Senadra's decay per key channel
+    """
+    import torch
+    from .. import ops
+    from ..config.spec import PartSpec
+    from ..engine.runner import StepContext, Workspace
+    from ..parts.experts import RoutedExperts
+    k = ops.kernels()
+    dev = torch.device("cuda:0")
+    bf = torch.bfloat16
+    nkv, md, hd, page = 8, 64, 128, 16
+    out = {}
+    hbm, tfl = peaks["hbm_gbs"], peaks["bf16_tflops"]
+
+    def mem_row(name, ms, nbytes):
+        out[name] = {"ms": ms, "gb_s": nbytes / ms / 1e6, "of_hbm_peak": nbytes / ms / 1e6 / hbm}
+
+    def flop_row(name, ms, flops):
+        out[name] = {"ms": ms, "tflops": flops / ms / 1e9, "of_bf16_peak": flops / ms / 1e9 / tfl}
+
+    diff = dict(num_heads=heads, num_kv_heads=nkv, k_dim=md, v_dim=hd, scale=0.125, softcap=30.0, lam=0.4, factor=0.6, eps=1e-6)
+    # ---- decode attention ---------------------------------------------------------------------------------------------------
+    for B, ctx in ((8, 4096), (64, 4096)):
+        meta, pages = _meta([ctx] * B, [1] * B, page, dev)
+        copies = [(torch.randn(pages, nkv, page, hd, device=dev).to(bf), torch.randn(pages, nkv, page, hd, device=dev).to(bf) * 0.3)
+                  for _ in range(2)]
+        q = torch.randn(B, heads * hd, device=dev).to(bf)
+        o = torch.empty(B, heads * hd, device=dev, dtype=bf)
+        ms = _timed([(lambda c=c: k.difference_attention(q, c[0], c[1], o, meta, **diff)) for c in copies])
+        mem_row(f"decode_attention_difference_{B}x{ctx}", ms, B * ctx * 2 * nkv * hd * 2)
+        q3 = q.view(B, heads, hd)
+        ms = _timed([(lambda c=c: k.paged_attention(q3, c[0], c[1], o, meta, num_heads=heads, num_kv_heads=nkv, head_dim=hd, scale=0.088,
+                                                    window=None)) for c in copies])
+        mem_row(f"decode_attention_qwen3_{B}x{ctx}", ms, B * ctx * 2 * nkv * hd * 2)
+        del copies
+    torch.cuda.empty_cache()
+    # ---- prefill attention: scores inside the polynomial's range, and scores up to the cap -------------------------------------
+    for T in (2048, 8192):
+        meta, pages = _meta([T], [T], page, dev)
+        kc = torch.randn(pages, nkv, page, hd, device=dev).to(bf)
+        vc = torch.randn(pages, nkv, page, hd, device=dev).to(bf) * 0.3
+        q = torch.randn(T, heads * hd, device=dev).to(bf)
+        o = torch.empty(T, heads * hd, device=dev, dtype=bf)
+        pairs = T * (T + 1) / 2
+        for tag, kw in (("", {}), ("_no_cap", {"softcap": None}), ("_to_the_cap", {"scale": 0.45}), ("_beyond_the_cap", {"scale": 1.5})):
+            ms = _timed([lambda: k.difference_attention(q, kc, vc, o, meta, **dict(diff, **kw))] * 3)
+            flop_row(f"prefill_attention_difference{tag}_{T}", ms, 4.0 * heads * (md + hd) * pairs)
+        q3 = q.view(T, heads, hd)
+        ms = _timed([lambda: k.paged_attention(q3, kc, vc, o, meta, num_heads=heads, num_kv_heads=nkv, head_dim=hd, scale=0.088,
+                                               window=None)] * 3)
+        flop_row(f"prefill_attention_qwen3_{T}", ms, 4.0 * heads * hd * pairs)
+        del kc, vc
+    torch.cuda.empty_cache()
+    # ---- rotation and cache write ------------------------------------------------------------------------------------------------
+    T = 2048
+    meta, pages = _meta([T], [T], page, dev)
+    slots = torch.arange(T, dtype=torch.int32, device=dev)
+    pos = torch.arange(T, dtype=torch.int32, device=dev)
+    wide = (heads + 2 * nkv) * hd
+    sets = [(torch.randn(T, wide, device=dev).to(bf), torch.empty(T, heads * hd, device=dev, dtype=bf),
+             torch.zeros(pages, nkv, page, hd, device=dev, dtype=bf), torch.zeros(pages, nkv, page, hd, device=dev, dtype=bf)) for _ in range(4)]
+    inv64 = torch.pow(torch.tensor(500000.0, dtype=torch.float64), -torch.arange(hd // 2, dtype=torch.float64) / (hd // 2)).to(dev)
+    table, table_half = torch.empty(T, hd // 2, 2, device=dev), torch.empty(T, md // 2, 2, device=dev)
+    k.rotary_table_scaled(inv64, pos, hd // 2, 1.0, table)
+    k.rotary_table_scaled(inv64, pos, md // 2, 1.0, table_half)
+    ms = _timed([(lambda t=t: k.rotate_pairs_store(t[0], 0, heads * hd, (heads + nkv) * hd, t[1], t[2], t[3], table_half, slots,
+                                                   num_heads=2 * heads, num_kv_heads=nkv, maps=2, k_dim=md, v_dim=hd, rot_dim=md)) for t in sets])
+    mem_row("rotate_pairs_store", ms, 2 * T * wide * 2)
+    ms = _timed([(lambda t=t: k.rotate_unit_store(t[0], 0, heads * hd, (heads + nkv) * hd, t[1].view(T, heads, hd), t[2], t[3], table, slots,
+                                                  num_heads=heads, num_kv_heads=nkv, k_dim=hd, v_dim=hd, rot_dim=hd, eps=1e-6,
+                                                  unit_norm=True)) for t in sets])
+    mem_row("rotate_unit_store_nogelorn", ms, 2 * T * wide * 2)
+    del sets
+    # ---- sum + norm ------------------------------------------------------------------------------------------------------------------
+    w, b = torch.ones(width, device=dev), torch.zeros(width, device=dev)
+    for n in (2048, 8):
+        sets = [(torch.randn(n, width, device=dev), torch.randn(n, width, device=dev).to(bf), torch.empty(n, width, device=dev, dtype=bf))
+                for _ in range(8)]
+        ms = _timed([(lambda t=t: k.tanh_add_tanh(t[0], t[1], 0.5, w, b, None, 0.5, w, b, t[2])) for t in sets])
+        mem_row(f"tanh_add_tanh_{n}", ms, n * width * (4 + 2 + 4 + 2))
+        ms = _timed([(lambda t=t: k.normed_add_rms_norm(t[0], t[1], w, 1e-6, None, w, 1e-6, t[2])) for t in sets])
+        mem_row(f"normed_add_rms_norm_nogelorn_{n}", ms, n * width * (4 + 2 + 4 + 2))
+        del sets
+    # ---- expert products ---------------------------------------------------------------------------------------------------------------
+    E, ff = 64, 1408
+    parts = {}
+    for name, params in (("corrected", {"top": 5, "activation": "relu2", "score": "softmax", "identity_experts": 4, "weight_scale": 1.5,
+                                        "intermediate_size": ff * 3 // 2, "shared_intermediate_size": ff * 3 // 2, "shared_gate": True}),
+                         ("softmax_nogelorn", {"top": 5, "activation": "silu", "score": "softmax_top", "intermediate_size": ff,
+                                               "shared_intermediate_size": ff})):
+        part = RoutedExperts(PartSpec("routed_experts", dict(params, hidden_size=width, num_experts=E, weight_on="output")), bf, dev)
+        # router weights such that the choices spread over the experts (and no correction, which would fix them)
+        std = {"router": 0.02, "correction": 0.0} if name == "corrected" else {"router": 1.0, "router.b": 1.0}
+        part.bind({tn: torch.randn(*ts.shape, device=dev).to(bf) * std.get(tn, 0.02) for tn, ts in part.tensors().items()})
+        parts[name] = part
+    for n in (2048, 8):
+        h = torch.randn(n, width, device=dev).to(bf)
+        for name, part in parts.items():
+            ctx_ = StepContext(Workspace(dev))
+            part.forward(h, ctx_)
+            ms = _timed(lambda: part.forward(h, ctx_))
+            ids = ctx_.buf("expert_ids", (n, part.top), torch.int32).flatten().tolist()
+            real = [i for i in ids if i < E]
+            if n >= 128:
+                flop_row(f"expert_feed_forward_{name}_{n}", ms, 2.0 * (len(real) + n) * 3 * ff * width)
+            else:
+                mem_row(f"expert_feed_forward_{name}_{n}", ms, (len(set(real)) + 1) * 3 * ff * width * 2)
+    del parts
+    torch.cuda.empty_cache()
+    # ---- the delta rule: one decay per head  vs  a decay per key channel ----------------------------------------------------------------
+    H, G, d, dv, taps = heads, heads // 2, 128, 128, 4
+    channels = 2 * G * d + H * dv
+    conv_w = torch.randn(channels, taps, device=dev) * 0.3
+    n_state = k.delta_state_floats(H, G, d, dv, taps)
+    ws = Workspace(dev)
+    norm_w = torch.ones(H * dv, device=dev)
+    for B, L in ((8, 1), (64, 1), (1, 2048), (4, 2048)):
+        n = B * L
+        sets = [(torch.randn(n, channels + H + H * dv, device=dev).to(bf) * 0.5, torch.randn(n, H * d, device=dev),
+                 torch.zeros(B, n_state, device=dev), torch.empty(n, H * dv, device=dev), torch.randn(n, 2 * H, device=dev))
+                for _ in range(4 if L == 1 else 1)]
+        sc = StepContext(ws)
+        sc.cu_q = torch.arange(0, n + 1, L, dtype=torch.int32, device=dev)
+        sc.state_slots = torch.arange(B, dtype=torch.int32, device=dev)
+        sc.seq_of_token = torch.arange(n, dtype=torch.int32, device=dev) // L
+        sc.max_q_len = L
+        size = dict(num_heads=H, num_kv_heads=G, dim=d, v_dim=dv)
+        a_log, dt_head, dt_channel = torch.zeros(H, device=dev), torch.zeros(H, device=dev), torch.zeros(H * d, device=dev)
+        for tag, fn in (("head", lambda t: k.delta_rule(t[0], 0, channels, t[4][:, :H], conv_w, a_log, dt_head, t[2], sc, t[3],
+                                                        b_pre=t[4][:, H:], **size)),
+                        ("channel_senadra", lambda t: k.delta_rule(t[0], 0, channels, t[1], conv_w, a_log, dt_channel, t[2], sc, t[3], **size))):
+            ms = _timed([(lambda t=t: fn(t)) for t in sets])
+            if L == 1:
+                mem_row(f"delta_rule_{tag}_decode_{B}", ms, B * 2 * H * d * dv * 4)
+            else:
+                flop_row(f"delta_rule_{tag}_prefill_{B}x{L}", ms, 6.0 * n * H * d * dv)
+        if (B, L) == (1, 2048):
+            gate = sets[0][0][:, channels + H:]
+            o16 = torch.empty(n, H * dv, device=dev, dtype=bf)
+            ms = _timed([lambda: k.head_norm_gate_act(sets[0][3], norm_w, gate, o16, num_heads=H, eps=1e-6, gate_act="silu")] * 4)
+            mem_row("head_norm_silu_gate", ms, n * H * dv * (4 + 2 + 2))
+        del sets
+    k.check_device_status()
+    return out
+
+
 def run_senadra(peaks: dict, width: int = 2048, heads: int = 16) -> dict:
     """The kernels of the Senadra design alone, each beside its like kernel of another path at equal size (16 heads of 128 on
     8 KV heads, chunks of 2,048 positions; recurrences of 16 value heads 128 x 128 on 8 query/key heads; latents of 512 + 64):

@@ -155,7 +155,37 @@ EQUAL_LEKILIX: Dict[str, dict] = {
     "n2k-moe": _lekilix_shape(2048, 16, experts=64, top=6, expert_ff=1408),
     "n4k-moe": _lekilix_shape(4096, 32, experts=64, top=6, expert_ff=2048),
 }
-DESIGN_SHAPES = {"galodra": GALODRA_SHAPES, "lekilix": LEKILIX_SHAPES, "senadra": SENADRA_SHAPES, "nogelorn": NOGELORN_SHAPES}
+
+
+def _ferodra_shape(width, heads, experts, identity, top, expert_ff, vocab=32768):
+    """Six layers of which the first two run twice (eight layer runs, as the shapes beside it): the delta rule (``heads`` value
+    heads 128 wide on half as many query/key heads 128 deep, four taps) and attention as the difference of two maps of 64 over
+    values of 128 on 8 key/value heads, in turn; experts without a gate -- one and a half times as wide as the gated ones
+    beside them, so that the weights are equal -- some identity outputs, and a shared expert."""
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": 8, "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "softcap": 30.0,
+                                          "diff": 0.4, "rot": {"dims": 64, "base": 1000000.0,
+                                                               "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    rec = {"type": "delta", "mixer": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}}
+    mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "identity": identity, "top": top, "scale": 1.5},
+           "shared": {"ff": expert_ff}}
+    return {"architecture": "Ferodra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "loop": {"start": 0, "stop": 2, "times": 2},
+            "layers": [dict(type=l["type"], mixer=copy.deepcopy(l["mixer"]), mlp=copy.deepcopy(mlp)) for l in (rec, att) * 3]}
+
+
+# Ferodra shapes with layer sizes of real models; beside each the Nogelorn shape of equal width, heads, layer runs and expert
+# weights (its closest relative: norms before and after, a looped stretch, recurrences beside attention, experts with a shared
+# one) and the Qwen3 dense shape of equal active size.
+FERODRA_SHAPES: Dict[str, dict] = {
+    "f2k-moe": _ferodra_shape(2048, 16, 64, 4, 5, 2112),
+    "f4k-moe": _ferodra_shape(4096, 32, 64, 4, 5, 3072),
+}
+EQUAL_NOGELORN = {"f2k-moe": "n2k-moe", "f4k-moe": "n4k-moe"}
+EQUAL_QWEN3.update({f: EQUAL_QWEN3[n] for f, n in EQUAL_NOGELORN.items()})
+DESIGN_SHAPES = {"galodra": GALODRA_SHAPES, "lekilix": LEKILIX_SHAPES, "senadra": SENADRA_SHAPES, "nogelorn": NOGELORN_SHAPES,
+                 "ferodra": FERODRA_SHAPES}
+# what each design is measured beside
+COMPARED_WITH = {"galodra": ("qwen3",), "lekilix": ("qwen3",), "senadra": ("qwen3",), "nogelorn": ("lekilix", "qwen3"),
+                 "ferodra": ("nogelorn", "qwen3")}
 FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "bf16_tflops_sustained": 1400.0}
 
 
@@ -203,10 +233,17 @@ def shape_config(name: str, layers: Optional[int] = None):
             raw["layers"] = raw["layers"][:layers]
             raw["loop"] = None if layers < raw["loop"]["stop"] else raw["loop"]
         return nogelorn_config_from_dict(raw)
+    if name in FERODRA_SHAPES:
+        from ..models.ferodra import ferodra_config_from_dict
+        raw = dict(FERODRA_SHAPES[name])
+        if layers:
+            raw["layers"] = raw["layers"][:layers]
+            raw["loop"] = None if layers < raw["loop"]["stop"] else raw["loop"]
+        return ferodra_config_from_dict(raw)
     try:
         raw = dict(SHAPES[name])
     except KeyError:
-        known = list(SHAPES) + list(GALODRA_SHAPES) + list(LEKILIX_SHAPES) + list(SENADRA_SHAPES) + list(NOGELORN_SHAPES)
+        known = list(SHAPES) + [n for shapes in DESIGN_SHAPES.values() for n in shapes]
         raise ValueError(f"unknown shape '{name}' ({' | '.join(known)})") from None
     if layers:
         raw["num_hidden_layers"] = layers
@@ -219,12 +256,19 @@ def random_model(name: str, dtype: str = "bfloat16", device="cuda:0", seed: int 
     from ..engine.model import Model
     cfg = shape_config(name, layers)
     arch = ("Galodra" if name in GALODRA_SHAPES else "Lekilix" if name in LEKILIX_SHAPES else "Senadra" if name in SENADRA_SHAPES
-            else "Nogelorn" if name in NOGELORN_SHAPES else "Qwen3ForCausalLM")
-    return Model.from_random(get_architecture(arch), cfg, seed=seed, dtype=dtype, device=device, norm_jitter=0.0)
+            else "Nogelorn" if name in NOGELORN_SHAPES else "Ferodra" if name in FERODRA_SHAPES else "Qwen3ForCausalLM")
+    model = Model.from_random(get_architecture(arch), cfg, seed=seed, dtype=dtype, device=device, norm_jitter=0.0)
+    if arch == "Ferodra":
+        # a norm by tanh does not bring a small stream to unit size: with rows of N(0, 0.02) every token would look alike to the
+        # routers and a whole batch would take the same few experts; rows of N(0, 1) spread them as trained rows do
+        model.embedding.weight.mul_(50.0)
+    return model
 
 
 def accounting_for(cfg, dtype_bytes: int = 2):
     """Bytes and flops of a step for a configuration of any built-in architecture."""
+    if type(cfg).__name__ == "FerodraConfig":
+        return FerodraAccounting(cfg, dtype_bytes)
     if type(cfg).__name__ == "NogelornConfig":
         return NogelornAccounting(cfg, dtype_bytes)
     if hasattr(cfg, "embedding_scale"):
@@ -422,6 +466,59 @@ class NogelornAccounting:
                 total += 2.0 * m.heads * (m.dim + m.vdim) * pairs
             for m in rec:
                 total += 4.0 * tokens * m.heads * m.dim * m.vdim               # the update and the read-out of every token
+        return total
+
+
+class FerodraAccounting:
+    """Bytes and flops of a Ferodra step, layer run by layer run (a layer of the looped stretch counts every time it runs).  A
+    decode step reads every dense weight once per run, of the experts those that the batch is expected to reach plus the shared
+    one, of a K/V cache every cell (both maps' keys and the values), and reads and writes every recurrence's float32 state.
+    A choice that falls on an identity output multiplies nothing."""
+
+    def __init__(self, cfg, dtype_bytes: int = 2):
+        self.cfg, self.b = cfg, dtype_bytes
+        self.head_w = cfg.vocab * cfg.width
+
+    def _layer(self, lc, batch: int):
+        """(weights read by a step of ``batch`` tokens, weights a token multiplies with) of one layer run."""
+        w, m = self.cfg.width, lc.mixer
+        if lc.type == "attention":
+            mix = w * (m.heads + m.kv_heads) * 2 * m.dim + w * m.kv_heads * m.vdim + m.heads * m.vdim * w
+        else:
+            mix = w * (2 * m.kv_heads * m.dim + 2 * m.heads * m.vdim + 2 * m.heads) + m.heads * m.vdim * w
+        f = lc.mlp
+        if f is None:
+            return mix, mix
+        if f.kind == "dense":
+            return mix + 3 * w * f.ff, mix + 3 * w * f.ff
+        outputs = f.experts + f.identity
+        reached = f.experts * (1.0 - (1.0 - f.top / outputs) ** batch)
+        fixed = w * (outputs + 1) + 2 * w * f.shared_ff
+        return mix + fixed + reached * 2 * w * f.ff, mix + fixed + f.top * f.experts / outputs * 2 * w * f.ff
+
+    def _runs(self):
+        return [self.cfg.layers[i] for i, _ in self.cfg.run_order()]
+
+    def decode_bytes(self, batch: int, ctx_avg: float) -> float:
+        total = self.head_w * self.b
+        for lc in self._runs():
+            total += self._layer(lc, batch)[0] * self.b
+            m = lc.mixer
+            if lc.type == "attention":
+                total += batch * ctx_avg * m.kv_heads * (2 * m.dim + m.vdim) * self.b
+            else:
+                total += batch * 2 * m.heads * m.dim * m.vdim * 4
+        return total
+
+    def prefill_flops(self, tokens: int) -> float:
+        total = 2.0 * self.head_w
+        for lc in self._runs():
+            m = lc.mixer
+            total += 2.0 * tokens * self._layer(lc, 1)[1]
+            if lc.type == "attention":
+                total += 2.0 * m.heads * 2 * (m.dim + m.vdim) * tokens * (tokens + 1) / 2
+            else:
+                total += 6.0 * tokens * m.heads * m.dim * m.vdim          # S^T k, the update and the read-out of every token
         return total
 
 
@@ -708,8 +805,8 @@ def serving_workload(shape: str = "0.6b", n_requests: int = 256, kv_cache_tokens
 # ---- one design beside another of equal size ------------------------------------------------------------------------
 def design_comparison(names: Sequence[str], batches: Sequence[int], prefill_tokens: Sequence[int], prompt_len: int, steps: int,
                       warmup: int, peaks: dict, device="cuda:0", cuda_graphs: bool = True, design: str = "galodra") -> dict:
-    """Decode and prefill throughput of each named shape of ``design`` and of the Qwen3 shape of equal size, random weights:
-    ``{name: {design: {...}, "qwen3": {...}}}`` with tokens/s and roofline fractions per point."""
+    """Decode and prefill throughput of each named shape of ``design`` and of the shapes of equal size it is measured beside
+    (``COMPARED_WITH``), random weights: ``{name: {design: {...}, "qwen3": {...}}}`` with tokens/s and roofline fractions per point."""
     import gc
     import torch
     from ..config.registry import get_architecture
@@ -718,9 +815,11 @@ def design_comparison(names: Sequence[str], batches: Sequence[int], prefill_toke
     out = {}
     for name in names:
         row = {}
-        for side in (design, "lekilix", "qwen3") if design == "nogelorn" else (design, "qwen3"):
+        for side in (design,) + COMPARED_WITH[design]:
             if side == design:
                 model = random_model(name, "bfloat16", device)
+            elif side == "nogelorn":
+                model = random_model(EQUAL_NOGELORN[name], "bfloat16", device)
             elif side == "lekilix":
                 from ..models.lekilix import lekilix_config_from_dict
                 model = Model.from_random(get_architecture("Lekilix"), lekilix_config_from_dict(EQUAL_LEKILIX[name]), seed=0,

@@ -27,8 +27,8 @@
 // The difference form (heads that are the difference of two softmax maps over the same values; see difference_attention.cu): a key
 // cell's halves are the two maps' keys and a query row's halves the two maps' queries, so a CTA owns 128 rows and its groups are
 // the MAPS: group m multiplies the half tiles m of Q and K, and both multiply their P with the same V.  Scores pass a tanh cap
-// before the softmax: as an odd polynomial of the score in packed float32 pairs where every |score| of a warp's rows in the tile
-// is within half the cap, else by the exponential and reciprocal units.  At the end the groups' outputs, which lie in the
+// before the softmax: as an odd polynomial of the score in packed float32 pairs, of degree 7 where every |score| of a warp's rows
+// in the tile is within half the cap, of degree 11 up to the cap, else by the exponential and reciprocal units.  At the end the groups' outputs, which lie in the
 // same lanes of tensor memory, are subtracted, each group taking one half of the columns.
 //
 // Every wait on an mbarrier is bounded: after kSpinLimit polls the waiter records where it gave up in
@@ -76,6 +76,7 @@ struct TcAttnParams {
     // difference form: t = cap_out * tanh(cap_in * s) takes the place of s (then scale_log2 is 1); cap_in 0: no cap
     float cap_in = 0.0f, cap_out = 0.0f;
     float cap_poly[4] = {0.0f, 0.0f, 0.0f, 0.0f};   // t = s (c0 + c1 s^2 + c2 s^4 + c3 s^6) for |s| <= cap_small
+    float cap_wide[6] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};      // the same of degree 11 for |s| <= 2 cap_small
     float cap_small = 0.0f;
     float lambda = 0.0f, factor = 0.0f, eps = 0.0f;
 };
@@ -474,6 +475,23 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
                             v[j] = __float_as_uint(y0);
                             v[j + 1] = __float_as_uint(y1);
                         }
+                    } else if (__all_sync(0xffffffffu, far <= 2.0f * p.cap_small)) {
+                        unsigned long long c[6];
+#pragma unroll
+                        for (int i2 = 0; i2 < 6; i2++) c[i2] = at_pack2(p.cap_wide[i2], p.cap_wide[i2]);
+#pragma unroll
+                        for (int j = 0; j < AT_BN; j += 2) {
+                            const unsigned long long x = at_pack2(__uint_as_float(v[j]), __uint_as_float(v[j + 1]));
+                            const unsigned long long x2 = at_mul2(x, x);
+                            unsigned long long y = at_fma2(x2, c[5], c[4]);
+#pragma unroll
+                            for (int i2 = 3; i2 >= 0; i2--) y = at_fma2(x2, y, c[i2]);
+                            y = at_mul2(x, y);
+                            float y0, y1;
+                            at_unpack2(y, y0, y1);
+                            v[j] = __float_as_uint(y0);
+                            v[j + 1] = __float_as_uint(y1);
+                        }
                     } else {
 #pragma unroll
                         for (int j = 0; j < AT_BN; j++) v[j] = __float_as_uint(p.cap_out * at_tanh(p.cap_in * __uint_as_float(v[j])));
@@ -835,13 +853,17 @@ IIAN_API int iian_attention_tc_difference(const void * q, const void * k_cache, 
     p.ld_q = (long long) nh * AT_HD;
     p.lambda = lambda; p.factor = factor; p.eps = eps;
     if (cap > 0.0f) {
-        // tanh(x) = x (a0 + a1 x^2 + a2 x^4 + a3 x^6) for |x| <= 1/2, fitted for the least largest error (1.3e-7 absolute)
-        static const double a[4] = {0.999997675672, -0.333206535381, 0.131451321517, -0.0433721740216};
+        // tanh(x) = x (a0 + a1 x^2 + ...), fitted for the least largest error: 1.3e-7 absolute up to 1/2, 2.4e-7 up to 1
+        static const double a[4] = {0.999997676142, -0.333206550541, 0.131451443375, -0.043372453431};
+        static const double w[6] = {0.999996853636, -0.333240033043, 0.132535224729, -0.050972798713, 0.016114115658, -0.00283944158113};
         const double c = (double) scale / cap, out_scale = (double) cap * 1.4426950408889634;
         p.cap_in = (float) c;
         p.cap_out = (float) out_scale;
         double f = out_scale * c;
-        for (int i = 0; i < 4; i++, f *= c * c) p.cap_poly[i] = (float) (f * a[i]);
+        for (int i = 0; i < 6; i++, f *= c * c) {
+            if (i < 4) p.cap_poly[i] = (float) (f * a[i]);
+            p.cap_wide[i] = (float) (f * w[i]);
+        }
         p.cap_small = (float) (0.5 / c);
     }
     const size_t smem = (size_t) 6 * AT_TILE_BYTES + 1024;
