@@ -66,6 +66,12 @@ struct AttnParams {
     int keep_first = 0;
     // one gate number per head instead of one per entry (rows of nh numbers): the head's size here, 0 otherwise
     int gate_per_head = 0;
+    // a cap on the scores: tanh(cap_in * s) takes the place of s, scale_log2 is cap * log2(e) and sink_to_raw 1 / cap; 0: no cap
+    float cap_in = 0.0f;
+    // fused form: the token's values are keep * v + share * first, rows of nkv * HD with ld_first elements between them; null: v
+    const __nv_bfloat16 * first = nullptr;
+    long long ld_first = 0;
+    float keep = 1.0f, share = 0.0f;
 };
 
 // first key of the chunk that position `pos` lies in
@@ -260,6 +266,13 @@ __global__ void __launch_bounds__(NW * 32, 3) attention_mma_kernel(const AttnPar
             }
             // ---- mask (only on tiles that touch a row's causal or window edge), online softmax ----
             const int key0 = phys(tile) * BN;
+            if (p.cap_in != 0.0f) {                         // the cap: from here on scores are in units of it
+#pragma unroll
+                for (int nt = 0; nt < BN / 8; nt++) {
+#pragma unroll
+                    for (int e = 0; e < 4; e++) sc[nt][e] = score_tanh(sc[nt][e] * p.cap_in);
+                }
+            }
             if (p.pen1 != nullptr) {                        // the distance penalty, in units of raw scores
 #pragma unroll
                 for (int nt = 0; nt < BN / 8; nt++) {
@@ -651,7 +664,18 @@ __global__ void __launch_bounds__(128, STAGES == 2 ? 3 : 2) attention_decode_ker
                         norm_rope(src, p.k_weight, tab != nullptr, s_new[0] + p0, s_new[0] + half + p0);
                     } else if (warp == 1) {
                         const __nv_bfloat16 * src = tok_in + (size_t) (p.nh + p.nkv + kvh) * HD;
-                        if (lane < CH) *reinterpret_cast<uint4 *>(s_new[1] + lane * 8) = *reinterpret_cast<const uint4 *>(src + lane * 8);
+                        if (lane < CH) {
+                            uint4 raw = *reinterpret_cast<const uint4 *>(src + lane * 8);
+                            if (p.first != nullptr) {
+                                float v[8], f[8];
+                                unpack8(raw, v);
+                                unpack8(*reinterpret_cast<const uint4 *>(p.first + (size_t) q0 * p.ld_first + (size_t) kvh * HD + lane * 8), f);
+#pragma unroll
+                                for (int c = 0; c < 8; c++) v[c] = mixed_value(v[c], f[c], p.keep, p.share);
+                                raw = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+                            }
+                            *reinterpret_cast<uint4 *>(s_new[1] + lane * 8) = raw;
+                        }
                     }
                 }
             }
@@ -715,6 +739,13 @@ __global__ void __launch_bounds__(128, STAGES == 2 ? 3 : 2) attention_decode_ker
                 mma16816(sc[1], qf[ks], b2, b3);
             }
             const int key0 = phys(tile_begin + i) * BN + warp * 16;
+            if (p.cap_in != 0.0f) {                         // the cap: from here on scores are in units of it
+#pragma unroll
+                for (int nt = 0; nt < 2; nt++) {
+#pragma unroll
+                    for (int e = 0; e < 4; e++) sc[nt][e] = score_tanh(sc[nt][e] * p.cap_in);
+                }
+            }
             if (p.pen1 != nullptr) {                        // the distance penalty, in units of raw scores
 #pragma unroll
                 for (int nt = 0; nt < 2; nt++) {
@@ -1080,6 +1111,13 @@ IIAN_API int iian_attention_decode_stages(int stages) {
     return IIAN_OK;
 }
 
+// scores in units of the cap from the hyperbolic tangent on
+static void set_cap(AttnParams & p, float scale, float cap) {
+    p.cap_in = scale / cap;
+    p.scale_log2 = cap * 1.4426950408889634f;
+    p.sink_to_raw = 1.0f / cap;
+}
+
 IIAN_API int iian_attention_mma_sink(
     const void * q, const void * k_cache, const void * v_cache, void * out, float * part_o, float * part_lse,
     int * counters, const int * cu_q, const int * ctx_len, const int * block_table, int max_blocks,
@@ -1122,6 +1160,14 @@ IIAN_API int iian_attention_mma_kept(
     const float * pen1, const float * pen2, const void * gate, long long ld_gate, int keep_first, int gate_per_head,
     cudaStream_t stream);
 
+IIAN_API int iian_attention_mma_capped(
+    const void * q, long long ld_q, const void * k_cache, const void * v_cache, void * out, float * part_o, float * part_lse,
+    int * counters, const int * cu_q, const int * ctx_len, const int * block_table, int max_blocks,
+    int N, int S, int max_q_len, int nh, int nkv, int hd, int page_size, int num_pages,
+    float scale, int window, int chunk, int n_split, int small_tiles, int * status, const float * sink,
+    const float * pen1, const float * pen2, const void * gate, long long ld_gate, int keep_first, int gate_per_head, float cap,
+    cudaStream_t stream);
+
 // The general entry.  q: rows of nh * hd with ld_q elements between them (a multiple of 8).  chunk > 0 (not together
 // with a window): key j is visible to position i iff j <= i and floor(i / chunk) == floor(j / chunk).  pen1, pen2:
 // f32 [nh] or both null: pen1[h] * ln(1 + pen2[h] * (i - j)) is taken off the scaled score (needs scale > 0).
@@ -1147,7 +1193,22 @@ IIAN_API int iian_attention_mma_kept(
     float scale, int window, int chunk, int n_split, int small_tiles, int * status, const float * sink,
     const float * pen1, const float * pen2, const void * gate, long long ld_gate, int keep_first, int gate_per_head,
     cudaStream_t stream) {
+    return iian_attention_mma_capped(q, ld_q, k_cache, v_cache, out, part_o, part_lse, counters, cu_q, ctx_len, block_table, max_blocks, N, S,
+                                     max_q_len, nh, nkv, hd, page_size, num_pages, scale, window, chunk, n_split, small_tiles, status, sink,
+                                     pen1, pen2, gate, ld_gate, keep_first, gate_per_head, 0.0f, stream);
+}
+
+// The same with a cap on the scores (0: none): cap * tanh(score / cap) takes the place of the scaled score (scale > 0; not together
+// with a penalty).
+IIAN_API int iian_attention_mma_capped(
+    const void * q, long long ld_q, const void * k_cache, const void * v_cache, void * out, float * part_o, float * part_lse,
+    int * counters, const int * cu_q, const int * ctx_len, const int * block_table, int max_blocks,
+    int N, int S, int max_q_len, int nh, int nkv, int hd, int page_size, int num_pages,
+    float scale, int window, int chunk, int n_split, int small_tiles, int * status, const float * sink,
+    const float * pen1, const float * pen2, const void * gate, long long ld_gate, int keep_first, int gate_per_head, float cap,
+    cudaStream_t stream) {
     if (N <= 0 || S <= 0) return IIAN_OK;
+    if (cap < 0.0f || (cap > 0.0f && (!(scale > 0.0f) || pen1 != nullptr))) return IIAN_ERR_SHAPE;
     if (keep_first < 0 || (keep_first > 0 && window <= 0)) return IIAN_ERR_SHAPE;
     if (sink != nullptr && !(scale > 0.0f)) return IIAN_ERR_SHAPE;
     if ((pen1 == nullptr) != (pen2 == nullptr) || (pen1 != nullptr && !(scale > 0.0f))) return IIAN_ERR_SHAPE;
@@ -1181,6 +1242,7 @@ IIAN_API int iian_attention_mma_kept(
     p.gate = (const __nv_bfloat16 *) gate; p.ld_gate = ld_gate;
     p.keep_first = keep_first;
     p.gate_per_head = gate != nullptr && gate_per_head ? hd : 0;
+    if (cap > 0.0f) set_cap(p, scale, cap);
     const int max_rows = max_q_len * (nh / nkv);
     int rc;
     if (p.keep_first > 0 || p.gate_per_head) {
@@ -1204,13 +1266,37 @@ IIAN_API int iian_attention_mma_kept(
 // new key and value to cache cell slots[i] (write_kv; a negative slot stores nothing), and attention over
 // the cache, in one launch.  Scratch as for iian_attention_mma's decode form; cluster != 0 (n_split 2..16)
 // needs none.  Up to 16 query heads per KV head.
+// With a sink, a cap and mixed values: iian_attention_decode_fused_mixed.
+IIAN_API int iian_attention_decode_fused_mixed(
+    const void * qkv, void * k_cache, void * v_cache, void * out, float * part_o, float * part_lse, int * counters,
+    const int * cu_q, const int * ctx_len, const int * block_table, int max_blocks,
+    int S, int nh, int nkv, int hd, int page_size, int num_pages, float scale, int window, int n_split, int cluster,
+    const float * q_weight, const float * k_weight, const float * table, const int * slots, float eps, int write_kv,
+    int * status, const float * sink, float cap, const void * first, long long ld_first, float keep, float share, cudaStream_t stream);
+
 IIAN_API int iian_attention_decode_fused(
     const void * qkv, void * k_cache, void * v_cache, void * out, float * part_o, float * part_lse, int * counters,
     const int * cu_q, const int * ctx_len, const int * block_table, int max_blocks,
     int S, int nh, int nkv, int hd, int page_size, int num_pages, float scale, int window, int n_split, int cluster,
     const float * q_weight, const float * k_weight, const float * table, const int * slots, float eps, int write_kv,
     int * status, cudaStream_t stream) {
+    return iian_attention_decode_fused_mixed(qkv, k_cache, v_cache, out, part_o, part_lse, counters, cu_q, ctx_len, block_table, max_blocks, S,
+                                             nh, nkv, hd, page_size, num_pages, scale, window, n_split, cluster, q_weight, k_weight, table,
+                                             slots, eps, write_kv, status, nullptr, 0.0f, nullptr, 0, 1.0f, 0.0f, stream);
+}
+
+// The same with a sink per head (f32 [nh] or null) in the denominator, a cap on the scores (0: none; both need scale > 0), and values
+// mixed before they are stored: keep * v + share * first, first: rows of nkv * hd bf16, ld_first (a multiple of 8) elements between
+// them, or null.
+IIAN_API int iian_attention_decode_fused_mixed(
+    const void * qkv, void * k_cache, void * v_cache, void * out, float * part_o, float * part_lse, int * counters,
+    const int * cu_q, const int * ctx_len, const int * block_table, int max_blocks,
+    int S, int nh, int nkv, int hd, int page_size, int num_pages, float scale, int window, int n_split, int cluster,
+    const float * q_weight, const float * k_weight, const float * table, const int * slots, float eps, int write_kv,
+    int * status, const float * sink, float cap, const void * first, long long ld_first, float keep, float share, cudaStream_t stream) {
     if (S <= 0) return IIAN_OK;
+    if (cap < 0.0f || ((cap > 0.0f || sink != nullptr) && !(scale > 0.0f))) return IIAN_ERR_SHAPE;
+    if (first != nullptr && ((ld_first & 7) || ((uintptr_t) first & 15))) return IIAN_ERR_ALIGN;
     if (nkv <= 0 || nh % nkv != 0 || nh / nkv > 16 || page_size <= 0 || n_split < 1) return IIAN_ERR_SHAPE;
     if (hd != 64 && hd != 128) return IIAN_ERR_SHAPE;
     const bool cl = cluster != 0 && n_split > 1;
@@ -1230,6 +1316,10 @@ IIAN_API int iian_attention_decode_fused(
     p.qkv = (const __nv_bfloat16 *) qkv; p.q_weight = q_weight; p.k_weight = k_weight;
     p.table = (const float2 *) table; p.slots = slots; p.eps = eps; p.write_kv = write_kv;
     p.status = status;
+    p.sink = sink;
+    p.sink_to_raw = sink != nullptr ? 1.0f / scale : 0.0f;
+    if (cap > 0.0f) set_cap(p, scale, cap);
+    p.first = (const __nv_bfloat16 *) first; p.ld_first = ld_first; p.keep = keep; p.share = share;
     const int max_rows = nh / nkv;
     if (cl) return hd == 128 ? launch_decode<128, true, true>(p, S, max_rows, stream) : launch_decode<64, true, true>(p, S, max_rows, stream);
     return hd == 128 ? launch_decode<128, false, true>(p, S, max_rows, stream) : launch_decode<64, false, true>(p, S, max_rows, stream);

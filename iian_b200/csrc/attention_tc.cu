@@ -31,6 +31,12 @@
 // in the tile is within half the cap, of degree 11 up to the cap, else by the exponential and reciprocal units.  At the end the groups' outputs, which lie in the
 // same lanes of tensor memory, are subtracted, each group taking one half of the columns.
 //
+// The capped form (plain heads whose scores pass a tanh cap, optionally with a sink): where the caller can bound the scores beforehand
+// (queries and keys that were normalised: |q . k| is at most the head's size times the largest product of their weights), the
+// polynomial's range is known before the launch and no score is looked at for it.  The cap rises with the score, so the maximum is
+// taken of the raw scores and capped alone, and the polynomial's last step x * P(x^2) is the multiply-add that takes the maximum off:
+// the cap costs four packed operations for two scores.
+//
 // Every wait on an mbarrier is bounded: after kSpinLimit polls the waiter records where it gave up in
 // `status`, and every role falls through to the common exit, where tensor memory is freed.
 #include <cuda.h>
@@ -73,11 +79,12 @@ struct TcAttnParams {
     int keep_first = 0;
     // one gate number per head (rows of nh numbers) instead of one per entry
     int gate_per_head = 0;
-    // difference form: t = cap_out * tanh(cap_in * s) takes the place of s (then scale_log2 is 1); cap_in 0: no cap
+    // difference and capped form: t = cap_out * tanh(cap_in * s) takes the place of s (then scale_log2 is 1); cap_in 0: no cap
     float cap_in = 0.0f, cap_out = 0.0f;
     float cap_poly[4] = {0.0f, 0.0f, 0.0f, 0.0f};   // t = s (c0 + c1 s^2 + c2 s^4 + c3 s^6) for |s| <= cap_small
     float cap_wide[6] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};      // the same of degree 11 for |s| <= 2 cap_small
     float cap_small = 0.0f;
+    int cap_range = 0;              // capped form: 1: every |s| <= cap_small, 2: <= 2 cap_small, 0: not known beforehand
     float lambda = 0.0f, factor = 0.0f, eps = 0.0f;
 };
 
@@ -207,13 +214,53 @@ __host__ __device__ constexpr unsigned at_idesc(int m, int n, bool b_mn) {
     return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn ? (1u << 16) : 0u) | ((unsigned) (n >> 3) << 17) | ((unsigned) (m >> 4) << 24);
 }
 
-// The form with kept first keys and a gate per head (AT_KEPT) and the difference form (AT_DIFF) are instances of their own, so that
-// the plain one stays as it was
-enum { AT_PLAIN = 0, AT_KEPT = 1, AT_DIFF = 2 };
+// t = s (c0 + c1 s^2 + ...) for one score
+template <int N> __device__ __forceinline__ float at_cap_one(float s, const float * c) {
+    const float x2 = s * s;
+    float y = c[N - 1];
+#pragma unroll
+    for (int i = N - 2; i >= 0; i--) y = fmaf(x2, y, c[i]);
+    return s * y;
+}
+// Two packed scores minus the maximum (neg2 = -max): x * (c0 + c1 x^2 + ...) + neg2
+template <int N> __device__ __forceinline__ unsigned long long at_cap_two(unsigned long long x, const unsigned long long * c, unsigned long long neg2) {
+    const unsigned long long x2 = at_mul2(x, x);
+    unsigned long long y = c[N - 1];
+#pragma unroll
+    for (int i = N - 2; i >= 0; i--) y = at_fma2(x2, y, c[i]);
+    return at_fma2(x, y, neg2);
+}
+
+// The form with kept first keys and a gate per head (AT_KEPT), the difference form (AT_DIFF) and the capped form (AT_CAP) are
+// instances of their own, so that the plain one stays as it was
+enum { AT_PLAIN = 0, AT_KEPT = 1, AT_DIFF = 2, AT_CAP = 3 };
+
+// probabilities of a row's 128 scores in v against the maximum -neg, capped by the polynomial of N coefficients: bf16 pairs into
+// v[0 .. 63], the sums in two packed pairs
+template <int N> __device__ __forceinline__ void at_capped_row(unsigned * v, const float * coef, float neg, unsigned long long * sum2) {
+    unsigned long long c[N];
+#pragma unroll
+    for (int i = 0; i < N; i++) c[i] = at_pack2(coef[i], coef[i]);
+    const unsigned long long neg2 = at_pack2(-neg, -neg);
+#pragma unroll
+    for (int j = 0; j < AT_BN; j += 4) {
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            const unsigned long long t = at_cap_two<N>(at_pack2(__uint_as_float(v[j + 2 * e]), __uint_as_float(v[j + 2 * e + 1])), c, neg2);
+            float t0, t1;
+            at_unpack2(t, t0, t1);
+            const float p0 = at_exp2(t0), p1 = at_exp2(t1);
+            sum2[e] = at_add2(sum2[e], at_pack2(p0, p1));
+            __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
+            v[(j >> 1) + e] = *reinterpret_cast<unsigned *>(&h);
+        }
+    }
+}
+
 template <int FORM>
 __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
     const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const TcAttnParams p) {
-    constexpr bool KEPT = FORM == AT_KEPT, DIFF = FORM == AT_DIFF;
+    constexpr bool KEPT = FORM == AT_KEPT, DIFF = FORM == AT_DIFF, CAP = FORM == AT_CAP;
     constexpr int CTA_ROWS = DIFF ? AT_BM : AT_ROWS;
     extern __shared__ __align__(1024) unsigned char at_smem_raw[];
     unsigned char * smem = (unsigned char *) (((uintptr_t) at_smem_raw + 1023) & ~(uintptr_t) 1023);
@@ -451,8 +498,18 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
 #pragma unroll
             for (int c0 = 0; c0 < AT_BN; c0 += 32) at_ld32(tS + lane_addr + (unsigned) c0, v + c0);
             at_wait_ld();
-            if constexpr (DIFF) {
-                if (p.cap_in > 0.0f) {                // t = cap_out tanh(cap_in s), of every column (hidden ones are set below)
+            // visible keys of this row in this tile: columns [lo, hi]; most tiles lie wholly below the diagonal
+            const int hi = row_ok ? min(AT_BN - 1, row_pos - key0) : -1;
+            int lo = p.window > 0 ? max(0, row_pos - p.window + 1 - key0) : max(0, row_lo - key0);
+            // kept first keys in this tile: columns [0, kept); where they reach the window's first column the row sees one
+            // stretch from column 0, else two (columns [kept, lo) stay hidden)
+            const int kept = KEPT ? max(0, p.keep_first - key0) : 0;
+            if (KEPT && kept >= lo) lo = 0;
+            const bool all_seen = __all_sync(0xffffffffu, lo <= 0 && hi >= AT_BN - 1);
+            // capped form, scores bounded beforehand, nothing hidden in this tile: the cap rides in the softmax's own arithmetic
+            const bool riding = CAP && p.cap_range != 0 && all_seen;
+            if constexpr (DIFF || CAP) {
+                if (p.cap_in > 0.0f && !riding) {     // t = cap_out tanh(cap_in s), of every column (hidden ones are set below)
                     float hi4[2] = {0.0f, 0.0f}, lo4[2] = {0.0f, 0.0f};
 #pragma unroll
                     for (int j = 0; j < AT_BN; j += 4) {
@@ -461,7 +518,8 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
                         hi4[1] = at_max3(hi4[1], __uint_as_float(v[j + 2]), __uint_as_float(v[j + 3]));
                         lo4[1] = at_min3(lo4[1], __uint_as_float(v[j + 2]), __uint_as_float(v[j + 3]));
                     }
-                    const float far = fmaxf(fmaxf(hi4[0], hi4[1]), -fminf(lo4[0], lo4[1]));
+                    float far = fmaxf(fmaxf(hi4[0], hi4[1]), -fminf(lo4[0], lo4[1]));
+                    if (CAP && p.cap_range != 0) far = 0.75f * (float) p.cap_range * p.cap_small;       // within the range's bound
                     if (__all_sync(0xffffffffu, far <= p.cap_small)) {
                         const unsigned long long c0 = at_pack2(p.cap_poly[0], p.cap_poly[0]), c1 = at_pack2(p.cap_poly[1], p.cap_poly[1]);
                         const unsigned long long c2 = at_pack2(p.cap_poly[2], p.cap_poly[2]), c3 = at_pack2(p.cap_poly[3], p.cap_poly[3]);
@@ -498,20 +556,13 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
                     }
                 }
             }
-            // visible keys of this row in this tile: columns [lo, hi]; most tiles lie wholly below the diagonal
-            const int hi = row_ok ? min(AT_BN - 1, row_pos - key0) : -1;
-            int lo = p.window > 0 ? max(0, row_pos - p.window + 1 - key0) : max(0, row_lo - key0);
-            // kept first keys in this tile: columns [0, kept); where they reach the window's first column the row sees one
-            // stretch from column 0, else two (columns [kept, lo) stay hidden)
-            const int kept = KEPT ? max(0, p.keep_first - key0) : 0;
-            if (KEPT && kept >= lo) lo = 0;
             if (p.pen1 != nullptr) {                // the distance penalty, in units of raw scores (masked keys are set below)
                 const float d0 = (float) (row_pos - key0);
 #pragma unroll
                 for (int j = 0; j < AT_BN; j++)
                     v[j] = __float_as_uint(fmaf(-pen_a, __log2f(fmaf(pen_b, d0 - (float) j, 1.0f)), __uint_as_float(v[j])));
             }
-            if (!__all_sync(0xffffffffu, lo <= 0 && hi >= AT_BN - 1)) {
+            if (!all_seen) {
                 if (two_sided) {
 #pragma unroll
                     for (int j = 0; j < AT_BN; j++)
@@ -530,7 +581,8 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
                 mx4[2] = at_max3(mx4[2], __uint_as_float(v[j + 4]), __uint_as_float(v[j + 5]));
                 mx4[3] = at_max3(mx4[3], __uint_as_float(v[j + 6]), __uint_as_float(v[j + 7]));
             }
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+            float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+            if (riding) mx = p.cap_range == 1 ? at_cap_one<4>(mx, p.cap_poly) : at_cap_one<6>(mx, p.cap_wide);
             // the maximum the sums are taken against moves only when it grew by more than 2^8 (or was unset)
             float corr = 1.0f;
             bool moved = false;
@@ -545,6 +597,10 @@ __global__ void __launch_bounds__(AT_THREADS, 1) attention_tc_kernel(
             // values have been used already
             const unsigned long long sl2 = at_pack2(sl, sl), neg2 = at_pack2(-neg, -neg);
             unsigned long long sum2[2] = {0ull, 0ull};
+            if (riding) {
+                if (p.cap_range == 1) at_capped_row<4>(v, p.cap_poly, neg, sum2);
+                else at_capped_row<6>(v, p.cap_wide, neg, sum2);
+            } else
 #pragma unroll
             for (int j = 0; j < AT_BN; j += 4) {
 #pragma unroll
@@ -716,6 +772,23 @@ static int at_make_map(CUtensorMap * map, const void * base, int num_pages, int 
     return r == CUDA_SUCCESS ? IIAN_OK : 2000 + (int) r;
 }
 
+// the cap's constants for scores s = q . k: t = cap * log2(e) * tanh(s * scale / cap)
+static void at_set_cap(TcAttnParams & p, float scale, float cap) {
+    // tanh(x) = x (a0 + a1 x^2 + ...), fitted for the least largest error: 1.3e-7 absolute up to 1/2, 2.4e-7 up to 1
+    static const double a[4] = {0.999997676142, -0.333206550541, 0.131451443375, -0.043372453431};
+    static const double w[6] = {0.999996853636, -0.333240033043, 0.132535224729, -0.050972798713, 0.016114115658, -0.00283944158113};
+    const double c = (double) scale / cap, out_scale = (double) cap * 1.4426950408889634;
+    p.cap_in = (float) c;
+    p.cap_out = (float) out_scale;
+    double f = out_scale * c;
+    for (int i = 0; i < 6; i++, f *= c * c) {
+        if (i < 4) p.cap_poly[i] = (float) (f * a[i]);
+        p.cap_wide[i] = (float) (f * w[i]);
+    }
+    p.cap_small = (float) (0.5 / c);
+    p.scale_log2 = 1.0f;
+}
+
 }  // namespace iian
 
 using namespace iian;
@@ -828,6 +901,47 @@ IIAN_API int iian_attention_tc_kept(const void * q, long long ld_q, const void *
     return iian_launch_status();
 }
 
+// The capped form: the plain one with cap * tanh(./cap) on the scaled scores (cap > 0, scale > 0), no chunks, penalty or gate.  bound: a
+// number no |score| before the cap exceeds, where the caller knows one, else 0.
+IIAN_API int iian_attention_tc_capped(const void * q, long long ld_q, const void * k_cache, const void * v_cache, void * out,
+                                      const int * cu_q, const int * ctx_len, const int * block_table, int max_blocks,
+                                      int N, int S, int max_q_len, int nh, int nkv, int hd, int page_size, int num_pages,
+                                      float scale, int window, float cap, float bound, int * status, const float * sink, cudaStream_t stream) {
+    if (N <= 0 || S <= 0) return IIAN_OK;
+    if (!(scale > 0.0f) || !(cap > 0.0f) || bound < 0.0f) return IIAN_ERR_SHAPE;
+    if (ld_q < (long long) nh * hd || (ld_q & 7)) return IIAN_ERR_ALIGN;
+    if (hd != AT_HD || nkv <= 0 || nh % nkv != 0 || window < 0) return IIAN_ERR_SHAPE;
+    if (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64 && page_size != 128) return IIAN_ERR_SHAPE;
+    if (status == nullptr) return IIAN_ERR_SHAPE;
+    if (((uintptr_t) q & 15) || ((uintptr_t) k_cache & 15) || ((uintptr_t) v_cache & 15) || ((uintptr_t) out & 15)) return IIAN_ERR_ALIGN;
+    if (S > 65535 || nkv > 65535) return IIAN_ERR_LIMIT;
+    CUtensorMap mk, mv;
+    int rc = at_make_map(&mk, k_cache, num_pages, nkv, page_size);
+    if (rc != IIAN_OK) return rc;
+    rc = at_make_map(&mv, v_cache, num_pages, nkv, page_size);
+    if (rc != IIAN_OK) return rc;
+    TcAttnParams p;
+    p.q = (const __nv_bfloat16 *) q; p.out = (__nv_bfloat16 *) out; p.cu_q = cu_q; p.ctx_len = ctx_len; p.block_table = block_table;
+    p.max_blocks = max_blocks; p.nh = nh; p.nkv = nkv; p.page_size = page_size; p.num_pages = num_pages; p.window = window;
+    p.status = status;
+    p.sink = sink;
+    p.sink_to_raw = 1.4426950408889634f;                     // capped scores are kept in units of log2
+    p.ld_q = ld_q;
+    at_set_cap(p, scale, cap);
+    p.cap_range = bound <= 0.0f ? 0 : bound <= 0.5f * cap ? 1 : bound <= cap ? 2 : 0;
+    const size_t smem = (size_t) 6 * AT_TILE_BYTES + 1024;
+    static bool configured = false;
+    if (!configured) {
+        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<AT_CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);
+        if (e != cudaSuccess) return 1000 + (int) e;
+        configured = true;
+    }
+    const int max_rows = max_q_len * (nh / nkv);
+    dim3 grid((max_rows + AT_ROWS - 1) / AT_ROWS, nkv, S);
+    attention_tc_kernel<AT_CAP><<<grid, AT_THREADS, smem, stream>>>(mk, mv, p);
+    return iian_launch_status();
+}
+
 // The difference form: q [N, nh, 2, 64], caches [num_pages, nkv, page_size, 128] (a key cell holds both maps' keys), out
 // [N, nh * 128].  Per map scores q . k * scale, then cap * tanh(./cap) (cap 0: as they are), causal, softmax; out = (map 1 - lambda
 // * map 2) / root mean square * factor.  scale > 0; page sizes and status as for the other forms.
@@ -852,20 +966,7 @@ IIAN_API int iian_attention_tc_difference(const void * q, const void * k_cache, 
     p.status = status;
     p.ld_q = (long long) nh * AT_HD;
     p.lambda = lambda; p.factor = factor; p.eps = eps;
-    if (cap > 0.0f) {
-        // tanh(x) = x (a0 + a1 x^2 + ...), fitted for the least largest error: 1.3e-7 absolute up to 1/2, 2.4e-7 up to 1
-        static const double a[4] = {0.999997676142, -0.333206550541, 0.131451443375, -0.043372453431};
-        static const double w[6] = {0.999996853636, -0.333240033043, 0.132535224729, -0.050972798713, 0.016114115658, -0.00283944158113};
-        const double c = (double) scale / cap, out_scale = (double) cap * 1.4426950408889634;
-        p.cap_in = (float) c;
-        p.cap_out = (float) out_scale;
-        double f = out_scale * c;
-        for (int i = 0; i < 6; i++, f *= c * c) {
-            if (i < 4) p.cap_poly[i] = (float) (f * a[i]);
-            p.cap_wide[i] = (float) (f * w[i]);
-        }
-        p.cap_small = (float) (0.5 / c);
-    }
+    if (cap > 0.0f) at_set_cap(p, scale, cap);
     const size_t smem = (size_t) 6 * AT_TILE_BYTES + 1024;
     static bool configured = false;
     if (!configured) {

@@ -28,7 +28,9 @@ BASE_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--shared", "-Xcompiler", "-fPIC
               "--expt-relaxed-constexpr"]
 SHARED_HEADERS = ["common.cuh"]
 # further headers that some sources share
-SOURCE_HEADERS: Dict[str, List[str]] = {"attention_mma": ["paged_mma.cuh"], "difference_attention_mma": ["paged_mma.cuh"]}
+SOURCE_HEADERS: Dict[str, List[str]] = {"attention_mma": ["paged_mma.cuh"], "difference_attention_mma": ["paged_mma.cuh"],
+                                         "moe": ["gated.cuh"], "postnorm": ["gated.cuh"], "gemm_stream": ["gated.cuh"],
+                                         "gemm_tcgen05": ["gated.cuh"]}
 
 # every library of the engine; build_all() compiles them all
 SOURCES = ["elementwise", "rope_kv", "attention_generic", "gemm_simt", "sampling", "gemm_skinny", "attention_mma", "prefetch", "gemm_tcgen05",

@@ -100,6 +100,9 @@ __device__ __forceinline__ float block_sum(float v, float * scratch) {
 __device__ __forceinline__ float rot_lo(float x, float y, float cs, float sn) { return __fmaf_rn(x, cs, -__fmul_rn(y, sn)); }
 __device__ __forceinline__ float rot_hi(float x, float y, float cs, float sn) { return __fmaf_rn(x, sn, __fmul_rn(y, cs)); }
 
+// A layer's value mixed with another layer's, spelled out for the same reason.
+__device__ __forceinline__ float mixed_value(float v, float first, float keep, float share) { return __fmaf_rn(share, first, __fmul_rn(keep, v)); }
+
 // 8 bf16 (16 bytes) -> 8 floats
 __device__ __forceinline__ void unpack8(const uint4 & raw, float * f) {
     const __nv_bfloat162 * p = reinterpret_cast<const __nv_bfloat162 *>(&raw);

@@ -37,13 +37,6 @@ struct DiffParams {
     int * status;                   // {code, where}, zero before the launch; null: cp.async instead of TMA
 };
 
-__device__ __forceinline__ float dm_tanh(float x) {
-    float e, r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));        // e^2x
-    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
-    return fmaf(-2.0f, r, 1.0f);
-}
-
 template <bool CLUSTER, int STAGES, bool TMA>
 __global__ void __launch_bounds__(128, STAGES == 2 ? 3 : 2) difference_decode_kernel(const DiffParams p, const __grid_constant__ KvMaps maps) {
     constexpr int NW = 4, BM = 16, HD = DM_HD;
@@ -230,7 +223,7 @@ __global__ void __launch_bounds__(128, STAGES == 2 ? 3 : 2) difference_decode_ke
             for (int nt = 0; nt < 4; nt++)
 #pragma unroll
                 for (int e = 0; e < 4; e++)
-                    sc[nt][e] = p.cap_in > 0.0f ? p.cap_log2 * dm_tanh(sc[nt][e] * p.cap_in) : sc[nt][e] * p.scale_log2;
+                    sc[nt][e] = p.cap_in > 0.0f ? p.cap_log2 * score_tanh(sc[nt][e] * p.cap_in) : sc[nt][e] * p.scale_log2;
             if (key0 + 31 > pos_min || !rows_full) {
 #pragma unroll
                 for (int nt = 0; nt < 4; nt++)

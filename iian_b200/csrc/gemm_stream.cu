@@ -18,6 +18,7 @@
 // and raises a flag in shared memory; every role then runs to the common exit without computing (the producer
 // first waits, bounded again, for the copies it has in flight).
 #include "common.cuh"
+#include "gated.cuh"
 
 namespace iian {
 
@@ -48,6 +49,8 @@ struct StreamExtra {                        // as SkinnyExtra of gemm_skinny.cu
     float * res;
     const float * norm_w;
     float * out_partial;
+    int act;                                // EPI 1: the gated activation (gated.cuh), `limit` for the clamped one
+    float limit;
 };
 
 __device__ __forceinline__ unsigned gs_smem(const void * p) { return (unsigned) __cvta_generic_to_shared(p); }
@@ -230,7 +233,7 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_stream_kernel(
 #pragma unroll
                     for (int wv = 0; wv < GS_WARPS; wv++) { gt += red[wv][r][n]; up += red[wv][r + 8][n]; }
                     if (scaled) { gt *= s_rs[n]; up *= s_rs[n]; }
-                    out[(size_t) n * (M / 2) + (m0 / 2 + f)] = from_f32<OutT>(gt / (1.0f + expf(-gt)) * up);
+                    out[(size_t) n * (M / 2) + (m0 / 2 + f)] = from_f32<OutT>(gated_value(gt, up, ex.act, ex.limit));
                 }
             }
         } else if (EPI == 2) {
@@ -355,26 +358,39 @@ IIAN_API int iian_gemm_stream_stages(int stages) {
 // norm_w) after res [B, M] float32 += bf16(product); out_partial [B, ceil(M / 16)] receives the sums of squares of res
 // per block of 16 rows of w.  status: two ints on the device, zero before the launch; non-zero afterwards means a wait
 // gave up and the output is not valid.  The results are those of iian_gemm_skinny_fused, bit for bit.
-IIAN_API int iian_gemm_stream(const void * x, const void * w, void * out, int out_dtype, int B, int M, int K, int epilogue,
-                              const float * in_partial, int in_tiles, float inv_width, float eps,
-                              float * res, const float * norm_w, float * out_partial, int * status, cudaStream_t stream) {
+static int gs_entry(const void * x, const void * w, void * out, int out_dtype, int B, int M, int K, int epilogue,
+                    const StreamExtra & ex, int * status, cudaStream_t stream) {
     if (B <= 0 || M <= 0) return IIAN_OK;
     if (B > 8) return IIAN_ERR_LIMIT;
     if (K <= 0 || K % 32 != 0) return IIAN_ERR_SHAPE;
     if (((uintptr_t) x & 15) || ((uintptr_t) w & 15)) return IIAN_ERR_ALIGN;
     if (status == nullptr) return IIAN_ERR_SHAPE;
-    if (in_partial != nullptr && in_tiles <= 0) return IIAN_ERR_SHAPE;
-    const StreamExtra ex = {in_partial, in_tiles, inv_width, eps, res, norm_w, out_partial};
+    if (ex.in_partial != nullptr && ex.in_tiles <= 0) return IIAN_ERR_SHAPE;
     if (epilogue == 1) {
         if (M % 16 != 0 || out_dtype != IIAN_BF16) return IIAN_ERR_SHAPE;
         return gs_launch_stages<1, __nv_bfloat16>(x, w, out, B, M, K, ex, status, stream);
     }
     if (epilogue == 2) {
-        if (out_dtype != IIAN_BF16 || res == nullptr || norm_w == nullptr || out_partial == nullptr) return IIAN_ERR_SHAPE;
+        if (out_dtype != IIAN_BF16 || ex.res == nullptr || ex.norm_w == nullptr || ex.out_partial == nullptr) return IIAN_ERR_SHAPE;
         return gs_launch_stages<2, __nv_bfloat16>(x, w, out, B, M, K, ex, status, stream);
     }
     if (epilogue != 0) return IIAN_ERR_SHAPE;
     if (out_dtype == IIAN_BF16) return gs_launch_stages<0, __nv_bfloat16>(x, w, out, B, M, K, ex, status, stream);
     if (out_dtype == IIAN_F32) return gs_launch_stages<0, float>(x, w, out, B, M, K, ex, status, stream);
     return IIAN_ERR_DTYPE;
+}
+
+IIAN_API int iian_gemm_stream(const void * x, const void * w, void * out, int out_dtype, int B, int M, int K, int epilogue,
+                              const float * in_partial, int in_tiles, float inv_width, float eps,
+                              float * res, const float * norm_w, float * out_partial, int * status, cudaStream_t stream) {
+    const StreamExtra ex = {in_partial, in_tiles, inv_width, eps, res, norm_w, out_partial, ACT_SILU, 0.0f};
+    return gs_entry(x, w, out, out_dtype, B, M, K, epilogue, ex, status, stream);
+}
+
+// Epilogue 1 with another gated activation than silu: act and limit as in gated.cuh.
+IIAN_API int iian_gemm_stream_gated(const void * x, const void * w, void * out, int B, int M, int K, int act, float limit, int * status,
+                                    cudaStream_t stream) {
+    if (act != ACT_SILU && act != ACT_CLAMPED && act != ACT_RELU) return IIAN_ERR_SHAPE;
+    const StreamExtra ex = {nullptr, 0, 0.0f, 0.0f, nullptr, nullptr, nullptr, act, limit};
+    return gs_entry(x, w, out, IIAN_BF16, B, M, K, 1, ex, status, stream);
 }

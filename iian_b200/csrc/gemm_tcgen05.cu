@@ -7,7 +7,7 @@
 // weights are stored in the file and in the reference (ggml_mul_mat(W, x), src/iian/graph.cpp:121-160).
 // The reference hands products of this size to cuBLAS (third_party/ggml/src/ggml-cuda/ggml-cuda.cu:
 // 1548-1608); this kernel is the engine's own, so that what follows the product can ride in its
-// epilogue: a plain store, or SiLU(gate) * up for a gate|up matrix whose rows are interleaved in groups
+// epilogue: a plain store, or SiLU(gate) * up (or another gated activation, gated.cuh) for a gate|up matrix whose rows are interleaved in groups
 // of 8 (gate rows 16j..16j+7, up rows 16j+8..16j+15 hold the same 8 features).
 //
 // Tile: 128 rows x BN columns (BN = 128 or 256), K in blocks of 64 (one 128-byte swizzle atom), STAGES
@@ -22,6 +22,7 @@
 #include <cuda.h>
 
 #include "common.cuh"
+#include "gated.cuh"
 
 namespace iian {
 
@@ -30,7 +31,8 @@ constexpr int TC_BK = 64;                 // 64 bf16 = 128 bytes = one swizzle a
 constexpr int TC_THREADS = 192;           // warp 0: TMA, warp 1: MMA + TMEM, warps 2..5: epilogue
 constexpr unsigned kSpinLimit = 2u * 1000u * 1000u;
 
-enum { EPI_STORE = 0, EPI_SWIGLU8 = 1, EPI_RESNORM = 2, EPI_RELU2 = 3 };      // EPI_RELU2 (grouped form): max(z, 0)^2
+enum { EPI_STORE = 0, EPI_SWIGLU8 = 1, EPI_RESNORM = 2, EPI_RELU2 = 3, EPI_GATED8 = 4 };      // EPI_RELU2 (grouped form): max(z, 0)^2;
+                                                  // EPI_GATED8: EPI_SWIGLU8 with the activation `act`
 
 struct TcStatus { int code; int where; };
 
@@ -55,6 +57,8 @@ struct TcExtra {
     const int * g_tiles;
     const int * g_offsets;
     int g_rows;
+    int act;                    // EPI_GATED8: the activation (gated.cuh), `limit` for the clamped one
+    float limit;
 };
 
 __device__ __forceinline__ unsigned smem_addr(const void * p) { return (unsigned) __cvta_generic_to_shared(p); }
@@ -128,7 +132,8 @@ __device__ __forceinline__ void mbar_arrive(unsigned bar) {
 // One accumulator tile (128 x BN, float32, in tensor memory) -> global memory.  `r` holds 32 consecutive
 // columns of this thread's row.
 template <int EPI, typename OutT>
-__device__ __forceinline__ void epilogue_store32(unsigned * r, OutT * __restrict__ out, int row, int col0, int N, int ldo, float rs) {
+__device__ __forceinline__ void epilogue_store32(unsigned * r, OutT * __restrict__ out, int row, int col0, int N, int ldo, float rs,
+                                                 int act, float limit) {
     if (rs != 1.0f) {
 #pragma unroll
         for (int i = 0; i < 32; i++) r[i] = __float_as_uint(__uint_as_float(r[i]) * rs);
@@ -174,7 +179,7 @@ __device__ __forceinline__ void epilogue_store32(unsigned * r, OutT * __restrict
 #pragma unroll
             for (int i = 0; i < 8; i++) {
                 const float g = __uint_as_float(r[16 * grp + i]), u = __uint_as_float(r[16 * grp + 8 + i]);
-                a[i] = g / (1.0f + __expf(-g)) * u;
+                a[i] = EPI == EPI_GATED8 ? gated_value_fast(g, u, act, limit) : g / (1.0f + __expf(-g)) * u;
             }
             if (col0 + 16 * grp + 16 <= N) {
                 if (sizeof(OutT) == 2 && (((uintptr_t) (dst + 8 * grp)) & 15) == 0) {
@@ -346,7 +351,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tcgen05_kernel(
                     if constexpr (EPI == EPI_RESNORM)
                         sq += epilogue_resnorm32(r, reinterpret_cast<__nv_bfloat16 *>(out), ex.res, ex.norm_w, row, n0 + c0, N, rs);
                     else
-                        epilogue_store32<EPI, OutT>(r, out, row, n0 + c0, N, ldo, rs);
+                        epilogue_store32<EPI, OutT>(r, out, row, n0 + c0, N, ldo, rs, ex.act, ex.limit);
                 }
             }
             if constexpr (EPI == EPI_RESNORM) {
@@ -524,7 +529,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TC_THREADS, 1) gemm_
                     if constexpr (EPI == EPI_RESNORM)
                         sq += epilogue_resnorm32(r, reinterpret_cast<__nv_bfloat16 *>(out), ex.res, ex.norm_w, row, n0 + c0, N, rs);
                     else
-                        epilogue_store32<EPI, OutT>(r, out, row, n0 + c0, N, ldo, rs);
+                        epilogue_store32<EPI, OutT>(r, out, row, n0 + c0, N, ldo, rs, ex.act, ex.limit);
                 }
             }
             if constexpr (EPI == EPI_RESNORM) {
@@ -641,7 +646,8 @@ static int tc_entry(const void * x, const void * w, void * out, int out_dtype, i
     if (T <= 0 || N <= 0) return IIAN_OK;
     if (K <= 0 || K % 8 != 0) return IIAN_ERR_SHAPE;
     if (((uintptr_t) x & 15) || ((uintptr_t) w & 15)) return IIAN_ERR_ALIGN;
-    if (epilogue == EPI_SWIGLU8 && N % 16 != 0) return IIAN_ERR_SHAPE;
+    const bool gated = epilogue == EPI_SWIGLU8 || epilogue == EPI_GATED8;
+    if (gated && N % 16 != 0) return IIAN_ERR_SHAPE;
     if (status == nullptr) return IIAN_ERR_SHAPE;
     if (bn != 128 && bn != 256 && bn != 512) return IIAN_ERR_SHAPE;
     if (ex.in_partial != nullptr && ex.in_tiles <= 0) return IIAN_ERR_SHAPE;
@@ -652,7 +658,13 @@ static int tc_entry(const void * x, const void * w, void * out, int out_dtype, i
     rc = make_map(&mb, w, N, K, pair ? 128 : bn);
     if (rc != IIAN_OK) return rc;
     TcStatus * st = (TcStatus *) status;
-    const int ldo = epilogue == EPI_SWIGLU8 ? N / 2 : N;
+    const int ldo = gated ? N / 2 : N;
+    if (epilogue == EPI_GATED8) {
+        if (out_dtype != IIAN_BF16) return IIAN_ERR_DTYPE;
+        if (pair) return launch_tc_pair<256, 3, 2, EPI_GATED8, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream);
+        if (bn == 256) return launch_tc<256, 4, EPI_GATED8, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream);
+        return launch_tc<128, 6, EPI_GATED8, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream);
+    }
     if (pair) {
         if (epilogue == EPI_RESNORM) {
             if (out_dtype != IIAN_BF16 || ex.res == nullptr || ex.norm_w == nullptr || ex.out_partial == nullptr) return IIAN_ERR_SHAPE;
@@ -687,16 +699,18 @@ static int tc_entry(const void * x, const void * w, void * out, int out_dtype, i
 }
 
 // The grouped product: x [T, K] bf16 with its rows sorted by group, w [groups * N, K] bf16 (group e's matrix in rows
-// e * N ..), out [T, N] or, with epilogue 1, [T, N / 2] (epilogue 3: max(z, 0)^2 of every entry); tiles = {row tiles, then (group, first row) per row tile of 128
+// e * N ..), out [T, N] or, with epilogue 1 or 4 (act and limit as in gated.cuh), [T, N / 2] (epilogue 3: max(z, 0)^2 of every entry); tiles = {row tiles, then (group, first row) per row tile of 128
 // rows}, offsets [groups + 1], both on the device; max_tiles bounds the row tiles (it sizes the grid).  bn: 128 or 256.
 IIAN_API int iian_gemm_tcgen05_grouped(const void * x, const void * w, void * out, int out_dtype, int T, int N, int groups, int K,
-                                       int epilogue, int bn, int * status, const int * tiles, const int * offsets, int max_tiles,
-                                       cudaStream_t stream) {
+                                       int epilogue, int act, float limit, int bn, int * status, const int * tiles, const int * offsets,
+                                       int max_tiles, cudaStream_t stream) {
     if (T <= 0 || N <= 0 || groups <= 0 || max_tiles <= 0) return IIAN_OK;
     if (K <= 0 || K % 8 != 0 || tiles == nullptr || offsets == nullptr || status == nullptr) return IIAN_ERR_SHAPE;
     if (((uintptr_t) x & 15) || ((uintptr_t) w & 15)) return IIAN_ERR_ALIGN;
-    if (epilogue != EPI_STORE && epilogue != EPI_SWIGLU8 && epilogue != EPI_RELU2) return IIAN_ERR_SHAPE;
-    if (epilogue == EPI_SWIGLU8 && N % 16 != 0) return IIAN_ERR_SHAPE;
+    const bool gated = epilogue == EPI_SWIGLU8 || epilogue == EPI_GATED8;
+    if (!gated && epilogue != EPI_STORE && epilogue != EPI_RELU2) return IIAN_ERR_SHAPE;
+    if (epilogue == EPI_GATED8 && act != ACT_SILU && act != ACT_CLAMPED && act != ACT_RELU) return IIAN_ERR_SHAPE;
+    if (gated && N % 16 != 0) return IIAN_ERR_SHAPE;
     if (bn != 128 && bn != 256) return IIAN_ERR_SHAPE;
     if (out_dtype != IIAN_BF16) return IIAN_ERR_DTYPE;
     if ((long long) groups * N > 2147483647LL) return IIAN_ERR_LIMIT;
@@ -706,8 +720,11 @@ IIAN_API int iian_gemm_tcgen05_grouped(const void * x, const void * w, void * ou
     rc = make_map(&mb, w, groups * N, K, bn);
     if (rc != IIAN_OK) return rc;
     TcStatus * st = (TcStatus *) status;
-    const int ldo = epilogue == EPI_SWIGLU8 ? N / 2 : N;
-    const TcExtra ex = {nullptr, 0, 0.0f, 0.0f, nullptr, nullptr, nullptr, tiles, offsets, N};
+    const int ldo = gated ? N / 2 : N;
+    const TcExtra ex = {nullptr, 0, 0.0f, 0.0f, nullptr, nullptr, nullptr, tiles, offsets, N, act, limit};
+    if (epilogue == EPI_GATED8)
+        return bn == 256 ? launch_tc<256, 4, EPI_GATED8, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream, max_tiles)
+                         : launch_tc<128, 6, EPI_GATED8, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream, max_tiles);
     if (epilogue == EPI_RELU2)
         return bn == 256 ? launch_tc<256, 4, EPI_RELU2, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream, max_tiles)
                          : launch_tc<128, 6, EPI_RELU2, __nv_bfloat16>(ma, mb, out, T, N, K, ldo, st, ex, stream, max_tiles);
@@ -725,7 +742,7 @@ IIAN_API int iian_gemm_tcgen05_grouped(const void * x, const void * w, void * ou
 // of a tile, 128 or 256; 512 runs tiles of 256 x 256 on pairs of SMs (tcgen05 cta_group::2).
 IIAN_API int iian_gemm_tcgen05(const void * x, const void * w, void * out, int out_dtype, int T, int N, int K, int epilogue,
                                int bn, int * status, cudaStream_t stream) {
-    if (epilogue == EPI_RESNORM) return IIAN_ERR_SHAPE;
+    if (epilogue == EPI_RESNORM || epilogue == EPI_GATED8) return IIAN_ERR_SHAPE;
     const TcExtra none = {nullptr, 0, 0.0f, 0.0f, nullptr, nullptr, nullptr};
     return tc_entry(x, w, out, out_dtype, T, N, K, epilogue, bn, status, none, stream);
 }
@@ -737,6 +754,18 @@ IIAN_API int iian_gemm_tcgen05(const void * x, const void * w, void * out, int o
 IIAN_API int iian_gemm_tcgen05_fused(const void * x, const void * w, void * out, int out_dtype, int T, int N, int K, int epilogue,
                                      int bn, int * status, const float * in_partial, int in_tiles, float inv_width, float eps,
                                      float * res, const float * norm_w, float * out_partial, cudaStream_t stream) {
+    if (epilogue == EPI_GATED8) return IIAN_ERR_SHAPE;
     const TcExtra ex = {in_partial, in_tiles, inv_width, eps, res, norm_w, out_partial};
     return tc_entry(x, w, out, out_dtype, T, N, K, epilogue, bn, status, ex, stream);
+}
+
+// The product over gate and up rows interleaved in groups of 8 with another gated activation than silu (act and limit as in
+// gated.cuh): out [T, N / 2] bf16.
+IIAN_API int iian_gemm_tcgen05_gated(const void * x, const void * w, void * out, int T, int N, int K, int act, float limit, int bn,
+                                     int * status, cudaStream_t stream) {
+    if (act != ACT_SILU && act != ACT_CLAMPED && act != ACT_RELU) return IIAN_ERR_SHAPE;
+    TcExtra ex = {};
+    ex.act = act;
+    ex.limit = limit;
+    return tc_entry(x, w, out, IIAN_BF16, T, N, K, EPI_GATED8, bn, status, ex, stream);
 }

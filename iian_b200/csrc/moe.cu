@@ -11,6 +11,7 @@
 // feed-forward can be recorded into a CUDA graph.  Every output element adds its products in the order k = 0, 1, ...,
 // and a token's expert outputs are added in the order of its choices, so a row's result does not depend on the batch.
 #include "common.cuh"
+#include "gated.cuh"
 
 namespace iian {
 
@@ -231,19 +232,6 @@ __global__ void moe_combine_mixed_kernel(const A * __restrict__ ys, const int * 
     }
 }
 
-// act 0: silu(g) * u; 1: gelu_tanh(g) * u; 2: with g' = min(g, limit), u' = clamp(u, -limit, limit):
-// g' sigmoid(1.702 g') (u' + 1)
-__device__ __forceinline__ float moe_gated(float g, float u, int act, float limit) {
-    if (act == 0) return g / (1.0f + expf(-g)) * u;
-    if (act == 2) {
-        g = fminf(g, limit);
-        u = fminf(fmaxf(u, -limit), limit);
-        return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
-    }
-    const float t = 0.7978845608028654f * (g + 0.044715f * g * g * g);
-    return 0.5f * g * (1.0f + tanhf(t)) * u;
-}
-
 // Rows [r0, r0 + rows) of x (sorted by expert) times expert e's weight block w[e] ([n_out, K], row-major):
 // out[r, m] = sum_k x[r, k] * w[e][m, k];  with GATED, w2[e] is a second block of the same shape and
 // out[r, m] = act(x . w[e][m]) * (x . w2[e][m]); without, act 3 squares the positive part; with GATED and w2 == w, an expert's block holds both, 2 n_out rows in
@@ -317,7 +305,7 @@ __global__ void __launch_bounds__(256) moe_grouped_gemm_kernel(const A * __restr
             if (m >= n_out) continue;
             float v = acc[i][j];
             // the gate and up products are rounded to the activation type first, as separate products would leave them
-            if (GATED) v = moe_gated(to_f32(from_f32<A>(v)), to_f32(from_f32<A>(acc2[i][j])), act, limit);
+            if (GATED) v = gated_value(to_f32(from_f32<A>(v)), to_f32(from_f32<A>(acc2[i][j])), act, limit);
             else if (act == 3) { v = fmaxf(v, 0.0f); v *= v; }
             out[(size_t) r * n_out + m] = from_f32<A>(v);
         }
@@ -427,10 +415,10 @@ IIAN_API int iian_moe_combine(const void * ys, const int * pos, void * out, int 
     return iian_moe_combine_weighted(ys, pos, nullptr, out, act_dtype, N, W, top, stream);
 }
 
-// x [M, K] sorted by expert; w (and w2, for the gated form) [E, n_out, K]; out [M, n_out]; act: 0 silu, 1 gelu (tanh); without
+// x [M, K] sorted by expert; w (and w2, for the gated form) [E, n_out, K]; out [M, n_out]; act: see gated.cuh; without
 // w2: 3 = max(z, 0)^2, anything else = the product as it is.
 // w2 == w: the gated form over blocks [E, 2 n_out, K] that hold both matrices interleaved in groups of 8 rows.
-// The plan's row tiles must be of iian_moe_tile_rows() rows.  act 2 (clamped, see moe_gated) takes `limit`.
+// The plan's row tiles must be of iian_moe_tile_rows() rows.  act: see gated.cuh; the clamped one takes `limit`.
 IIAN_API int iian_moe_grouped_gemm_act(const void * x, const void * w, const void * w2, void * out, const int * offsets,
                                        const int * tiles, int max_tiles, int act_dtype, int w_dtype, int n_out, int K, int act,
                                        float limit, cudaStream_t stream) {

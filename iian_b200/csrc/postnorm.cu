@@ -7,9 +7,10 @@
 //   gated_add_layer_norm:  s = alpha * x + sub * sigmoid(g + gb);   y = (s - mean(s)) / sqrt(var(s) + eps) * w + b
 //                          with var the mean of the squared deviations (two passes over the row, held in shared memory)
 //   depth_mix:             y[r] = sum_j c[j] * X_j[row_j(r)]   in the order j = 0, 1, 2, ...
-//   gated_act:             y = act(gate) * up,  act = silu (z / (1 + exp(-z))) or the tanh form of gelu
-//                          (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))))
+//   gated_act:             y = act(gate) * up,  act = silu (z / (1 + exp(-z))), the tanh form of gelu
+//                          (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))), the positive part, or the clamped form (gated.cuh)
 #include "common.cuh"
+#include "gated.cuh"
 
 namespace iian {
 
@@ -193,12 +194,6 @@ __global__ void depth_mix_kernel(MixTerms terms, int n_terms, const float * __re
     }
 }
 
-__device__ __forceinline__ float act_apply(float z, int act) {
-    if (act == 0) return z / (1.0f + expf(-z));
-    const float t = 0.7978845608028654f * (z + 0.044715f * z * z * z);
-    return 0.5f * z * (1.0f + tanhf(t));
-}
-
 // in rows: [gate (F) | up (F)] (interleave 0) or groups of 16 columns holding 8 gate values and then the 8 up
 // values of the same features (interleave 8); row stride ld_in elements
 template <typename A>
@@ -212,14 +207,7 @@ __global__ void gated_act_kernel(const A * __restrict__ in, long long ld_in, A *
     const int col = (int) (idx - r * F);
     const size_t gi = r * ld_in + (interleave ? (size_t) (col / 8) * 16 + col % 8 : (size_t) col);
     const size_t ui = interleave ? gi + 8 : gi + F;
-    float g = to_f32(in[gi]), u = to_f32(in[ui]);
-    if (act == 2) {     // clamped: g' = min(g, limit), u' = clamp(u, -limit, limit); g' sigmoid(1.702 g') (u' + 1)
-        g = fminf(g, limit);
-        u = fminf(fmaxf(u, -limit), limit);
-        out[idx] = from_f32<A>(g / (1.0f + expf(-1.702f * g)) * (u + 1.0f));
-        return;
-    }
-    out[idx] = from_f32<A>(act_apply(g, act) * u);
+    out[idx] = from_f32<A>(gated_value(to_f32(in[gi]), to_f32(in[ui]), act, limit));
 }
 
 }  // namespace iian
@@ -298,11 +286,11 @@ IIAN_API int iian_gated_act(const void * in, long long ld_in, void * out, int ac
     return iian_gated_act_limit(in, ld_in, out, act_dtype, N, F, interleave, act, 0.0f, stream);
 }
 
-// act: 0 silu, 1 gelu (tanh form), 2 clamped (takes `limit`)
+// act: 0 silu, 1 gelu (tanh form), 2 clamped (takes `limit`), 4 the positive part
 IIAN_API int iian_gated_act_limit(const void * in, long long ld_in, void * out, int act_dtype, int N, int F, int interleave, int act,
                                   float limit, cudaStream_t stream) {
     if (interleave != 0 && (interleave != 8 || F % 8 != 0)) return IIAN_ERR_SHAPE;
-    if (act < 0 || act > 2) return IIAN_ERR_SHAPE;
+    if (act != ACT_SILU && act != ACT_GELU_TANH && act != ACT_CLAMPED && act != ACT_RELU) return IIAN_ERR_SHAPE;
     const size_t total = (size_t) N * F;
     if (total == 0) return IIAN_OK;
     const int threads = 256;

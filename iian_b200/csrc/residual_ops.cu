@@ -9,7 +9,10 @@
 //   relu2                 max(z, 0)^2
 //   tanh_cap              z <- cap * tanh(z / cap), in place
 //   normed_add_rms_norm   x += y / sqrt(mean(y^2) + eps_y) * u [+ e]  (a sub-layer output that passes a norm of its own before
-//                         it joins the stream; e: a second float32 addend);  out = x / sqrt(mean(x^2) + eps) * w    (each optional)
+//                         it joins the stream; e: a second float32 addend);  out = x / sqrt(mean(x^2) + eps) * w    (each optional);
+//                         with out and without w: out = x, the stream as it is in the activation type
+//   embedding_placed      x = a E[token] [+ P[position]];  x <- x / sqrt(mean(x^2) + eps) * w;  copy = x in the activation type
+//                         (P, w, copy optional)
 //
 // `A` is the activation type; sums, norms and the stream are float32.  A row's result depends on that row only.
 #include "common.cuh"
@@ -326,6 +329,10 @@ __global__ void normed_add_rms_norm_kernel(float * __restrict__ residual, const 
         ss = fmaf(v, v, ss);
     }
     if (out == nullptr) return;
+    if (weight == nullptr) {                                 // (a thread reads back what it wrote itself)
+        for (int i = threadIdx.x; i < H; i += blockDim.x) out[base + i] = from_f32<A>(r[i]);
+        return;
+    }
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float) H + eps);
     for (int i = threadIdx.x; i < H; i += blockDim.x) out[base + i] = from_f32<A>(r[i] * inv * weight[i]);
@@ -379,11 +386,12 @@ __global__ void normed_add_rms_norm_vec_kernel(float * __restrict__ residual, co
                 v[k].x += e4.x; v[k].y += e4.y; v[k].z += e4.z; v[k].w += e4.w;
             }
             if (y != nullptr || extra != nullptr) store4(residual + base + i, v[k]);
+            if (out != nullptr && weight == nullptr) store4(out + base + i, v[k]);
         }
         ss = fmaf(v[k].x, v[k].x, ss); ss = fmaf(v[k].y, v[k].y, ss);
         ss = fmaf(v[k].z, v[k].z, ss); ss = fmaf(v[k].w, v[k].w, ss);
     }
-    if (out == nullptr) return;
+    if (out == nullptr || weight == nullptr) return;
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float) H + eps);
 #pragma unroll
@@ -392,6 +400,82 @@ __global__ void normed_add_rms_norm_vec_kernel(float * __restrict__ residual, co
         if (i < H) {
             const float4 w4 = load4(weight + i);
             store4(out + base + i, make_float4(v[k].x * inv * w4.x, v[k].y * inv * w4.y, v[k].z * inv * w4.z, v[k].w * inv * w4.w));
+        }
+    }
+}
+
+// ---- where the stream starts: a token's row, its position's row, a norm ---------------------------------------------------
+// T: the tables' type (both the same); a block per token.  Rows outside the tables are taken at their ends.
+template <typename T, typename A>
+__global__ void embedding_placed_kernel(const T * __restrict__ table, const int * __restrict__ tokens, float scale,
+                                        const T * __restrict__ places, const int * __restrict__ positions,
+                                        const float * __restrict__ weight, float eps, float * __restrict__ x, A * __restrict__ copy, int H,
+                                        int V, int P) {
+    pdl_wait();
+    pdl_launch_dependents();
+    __shared__ float scratch[32];
+    const size_t t = blockIdx.x, base = t * H;
+    const T * e = table + (size_t) min(max(tokens[t], 0), V - 1) * H;
+    const T * p = places != nullptr ? places + (size_t) min(max(positions[t], 0), P - 1) * H : nullptr;
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float v = p != nullptr ? fmaf(to_f32(e[i]), scale, to_f32(p[i])) : to_f32(e[i]) * scale;
+        x[base + i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    float inv = 1.0f;
+    if (weight != nullptr) {
+        ss = block_sum(ss, scratch);
+        inv = 1.0f / sqrtf(ss / (float) H + eps);
+    }
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {      // (each thread its own entries again)
+        const float v = weight != nullptr ? x[base + i] * inv * weight[i] : x[base + i];
+        x[base + i] = v;
+        if (copy != nullptr) copy[base + i] = from_f32<A>(v);
+    }
+}
+
+template <typename T, typename A>
+__global__ void embedding_placed_vec_kernel(const T * __restrict__ table, const int * __restrict__ tokens, float scale,
+                                            const T * __restrict__ places, const int * __restrict__ positions,
+                                            const float * __restrict__ weight, float eps, float * __restrict__ x, A * __restrict__ copy,
+                                            int H, int V, int P) {
+    pdl_wait();
+    pdl_launch_dependents();
+    __shared__ float scratch[32];
+    const size_t t = blockIdx.x, base = t * H;
+    const T * e = table + (size_t) min(max(tokens[t], 0), V - 1) * H;
+    const T * p = places != nullptr ? places + (size_t) min(max(positions[t], 0), P - 1) * H : nullptr;
+    float4 v[kRowKeep];
+    float ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < kRowKeep; k++) {
+        const int i = 4 * (threadIdx.x + k * blockDim.x);
+        v[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (i < H) {
+            const float4 a = load4(e + i);
+            float4 b = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (p != nullptr) b = load4(p + i);
+            v[k] = make_float4(fmaf(a.x, scale, b.x), fmaf(a.y, scale, b.y), fmaf(a.z, scale, b.z), fmaf(a.w, scale, b.w));
+        }
+        ss = fmaf(v[k].x, v[k].x, ss); ss = fmaf(v[k].y, v[k].y, ss);
+        ss = fmaf(v[k].z, v[k].z, ss); ss = fmaf(v[k].w, v[k].w, ss);
+    }
+    float inv = 1.0f;
+    if (weight != nullptr) {
+        ss = block_sum(ss, scratch);
+        inv = 1.0f / sqrtf(ss / (float) H + eps);
+    }
+#pragma unroll
+    for (int k = 0; k < kRowKeep; k++) {
+        const int i = 4 * (threadIdx.x + k * blockDim.x);
+        if (i < H) {
+            if (weight != nullptr) {
+                const float4 w4 = load4(weight + i);
+                v[k] = make_float4(v[k].x * inv * w4.x, v[k].y * inv * w4.y, v[k].z * inv * w4.z, v[k].w * inv * w4.w);
+            }
+            store4(x + base + i, v[k]);
+            if (copy != nullptr) store4(copy + base + i, v[k]);
         }
     }
 }
@@ -527,12 +611,12 @@ IIAN_API int iian_tanh_cap(float * x, float cap, long long total, cudaStream_t s
 }
 
 // residual: f32 [N, H] in place; y: A [N, H] or null; u: f32 [H] or null (y joins the stream as it is); extra: f32 [N, H] or
-// null; weight f32 [H] and out A [N, H]: both or neither.
+// null; out A [N, H] or null: the normalised stream with weight f32 [H], the stream itself without.
 IIAN_API int iian_normed_add_rms_norm(float * residual, const void * y, const float * u, float eps_y, const float * extra,
                                       const float * weight, void * out, int act_dtype, int N, int H, float eps,
                                       cudaStream_t stream) {
     if (N <= 0) return IIAN_OK;
-    if (H <= 0 || (out != nullptr && weight == nullptr)) return IIAN_ERR_SHAPE;
+    if (H <= 0) return IIAN_ERR_SHAPE;
     if (act_dtype != IIAN_F32 && act_dtype != IIAN_BF16) return IIAN_ERR_DTYPE;
     if (const int vt = row_vec_threads(H, act_dtype == IIAN_F32 ? 4 : 2, {y, out}, {residual, u, extra, weight})) {
         if (act_dtype == IIAN_F32)
@@ -547,4 +631,29 @@ IIAN_API int iian_normed_add_rms_norm(float * residual, const void * y, const fl
                            eps_y, extra, weight, (float *) out, H, eps);
     return iian_launch(normed_add_rms_norm_kernel<__nv_bfloat16>, dim3(N), dim3(threads), 0, stream, residual,
                        (const __nv_bfloat16 *) y, u, eps_y, extra, weight, (__nv_bfloat16 *) out, H, eps);
+}
+
+// table T [V, H], places T [P, H] or null (then positions is not read), tokens and positions i32 [N], weight f32 [H] or null (no
+// norm), x f32 [N, H], copy A [N, H] or null.
+IIAN_API int iian_embedding_placed(const void * table, const void * places, int table_dtype, const int * tokens, const int * positions,
+                                   float scale, const float * weight, float eps, float * x, void * copy, int act_dtype, int N, int H,
+                                   int V, int P, cudaStream_t stream) {
+    if (N <= 0) return IIAN_OK;
+    if (H <= 0 || V <= 0 || (places != nullptr && (P <= 0 || positions == nullptr))) return IIAN_ERR_SHAPE;
+    typedef __nv_bfloat16 bf;
+    const int tb = table_dtype == IIAN_F32 ? 4 : 2, ab = act_dtype == IIAN_F32 ? 4 : 2;
+    int vt = row_vec_threads(H, ab, {copy}, {x, weight});
+    if ((uintptr_t) table % (4 * tb) || (uintptr_t) places % (4 * tb)) vt = 0;
+    const int threads = vt ? vt : H >= 1024 ? 256 : 128;
+#define IIAN_PLACED(T, A)                                                                                                          \
+    return vt ? iian_launch(embedding_placed_vec_kernel<T, A>, dim3(N), dim3(threads), 0, stream, (const T *) table, tokens, scale, \
+                            (const T *) places, positions, weight, eps, x, (A *) copy, H, V, P)                                     \
+              : iian_launch(embedding_placed_kernel<T, A>, dim3(N), dim3(threads), 0, stream, (const T *) table, tokens, scale,     \
+                            (const T *) places, positions, weight, eps, x, (A *) copy, H, V, P)
+    if (table_dtype == IIAN_F32 && act_dtype == IIAN_F32) IIAN_PLACED(float, float);
+    if (table_dtype == IIAN_BF16 && act_dtype == IIAN_BF16) IIAN_PLACED(bf, bf);
+    if (table_dtype == IIAN_F32 && act_dtype == IIAN_BF16) IIAN_PLACED(float, bf);
+    if (table_dtype == IIAN_BF16 && act_dtype == IIAN_F32) IIAN_PLACED(bf, float);
+#undef IIAN_PLACED
+    return IIAN_ERR_DTYPE;
 }

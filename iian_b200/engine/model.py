@@ -114,6 +114,8 @@ class Model:
                 block.bound()
         if getattr(self.head, "tied", False):
             self.head.tie(self.embedding.weight)
+        if getattr(self.head, "scale", 1.0) != 1.0:
+            self.final_norm.absorb_factor(self.head.scale)         # a factor on the logits is one on the rows the head reads
         self.vocab_size = self.spec.vocab_size
         self.hidden_size = self.spec.hidden_size
         self.max_position = self.spec.max_position

@@ -135,12 +135,13 @@ def supports(model) -> bool:
     from ..parts.position import NoPosition, Rotary
     if model.device.type != "cuda" or type(model.embedding) is not TokenEmbedding or type(model.head) is not LMHead \
             or type(model.final_norm) is not RMSNorm or model.embedding.scale != 1.0 or model.stream_parts \
-            or model.embedding.side_width or model.head.softcap is not None:
+            or model.embedding.side_width or model.embedding.positions or model.embedding.norm is not None \
+            or model.head.softcap is not None or model.head.scale != 1.0:
         return False
     for blk in model.blocks:
         if type(blk) is not PreNormResidualBlock or type(blk.mixer) is not Attention or type(blk.feed_forward) is not GatedMLP \
                 or type(blk.mixer_norm) is not RMSNorm or type(blk.feed_forward_norm) is not RMSNorm \
-                or type(blk.mixer.position) not in (Rotary, NoPosition):
+                or type(blk.mixer.position) not in (Rotary, NoPosition) or blk.feed_forward.activation != "silu":
             return False
     return True
 

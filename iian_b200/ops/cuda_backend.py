@@ -279,11 +279,7 @@ class CudaKernels:
     _stream_stages_set = None
 
     def _gemm_stream(self, x, w, out, n, m, k, epilogue, in_p=0, in_tiles=0, inv_w=0.0, eps=0.0, res=0, nw=0, out_p=0) -> None:
-        if self._stream_stages_set != self.STREAM_STAGES:
-            fn = _fn("gemm_stream", "iian_gemm_stream_stages", [c_int])
-            if fn(self.STREAM_STAGES) != 0:
-                raise KernelError("gemm_stream: the ring has 6 or 12 stages")
-            type(self)._stream_stages_set = self.STREAM_STAGES
+        self._apply_stream_stages()
         status = self.tcgen05_status_buffer(x.device).data_ptr()
         CudaKernels._tc_used = True
         fn = _fn("gemm_stream", "iian_gemm_stream",
@@ -330,6 +326,55 @@ class CudaKernels:
         """Whether ``linear_swiglu`` can run for these operands (else: linear, then swiglu)."""
         n, k = x.shape
         return interleave == 8 and w.shape[0] % 16 == 0 and (self._tcgen05_ok(x, w, n, k) or self._skinny_ok(x, w, n, k))
+
+    def can_fuse_gated(self, x: torch.Tensor, w: torch.Tensor, interleave: int, activation: str) -> bool:
+        """Whether ``linear_gated`` can run for these operands (else: linear, then gated_act)."""
+        n, k = x.shape
+        return (activation in ("silu", "clamped_swish", "relu") and interleave == 8 and w.shape[0] % 16 == 0
+                and (self._tcgen05_ok(x, w, n, k) or (self.STREAM_PRODUCT and self._skinny_ok(x, w, n, k))))
+
+    def linear_gated(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, activation: str, limit: float = 0.0) -> None:
+        """out[t, f] = act(x . w_gate_f, x . w_up_f) for w with gate and up rows interleaved in groups of 8 (activations as in
+        ``gated_act``): the activation rides in the product's epilogue."""
+        n, k = x.shape
+        m = w.shape[0]
+        if out.shape != (n, m // 2) or w.shape[1] != k or out.dtype != torch.bfloat16:
+            raise KernelError(f"linear_gated: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)} do not fit")
+        status = self.tcgen05_status_buffer(x.device).data_ptr()
+        CudaKernels._tc_used = True
+        act = self.ACTIVATIONS[activation]
+        if self._tcgen05_ok(x, w, n, k):
+            fn = _fn("gemm_tcgen05", "iian_gemm_tcgen05_gated",
+                     [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p])
+            _check(fn(_cuda(x, "linear x"), _cuda(w, "linear w"), _cuda(out, "linear out"), n, m, k, act, limit,
+                      self.tcgen05_tile(n, m), status, _stream()), "gemm_tcgen05_gated")
+            return
+        if not self._skinny_ok(x, w, n, k):
+            raise KernelError("linear_gated: up to 8 rows of bfloat16 with K a multiple of 32, or the tcgen05 kernel's range")
+        self._before_streaming_product(x, w)
+        fn = _fn("gemm_stream", "iian_gemm_stream_gated",
+                 [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
+        _check(fn(_cuda(x, "linear x"), _cuda(w, "linear w"), _cuda(out, "linear out"), n, m, k, act, limit, status, _stream()),
+               "gemm_stream_gated")
+        self._after_streaming_product(w)
+
+    def _before_streaming_product(self, x, w) -> None:
+        if self.prefetcher is not None:
+            self.prefetcher.before_product(self)
+        self._apply_stream_stages()
+
+    def _after_streaming_product(self, w) -> None:
+        if self.weight_log is not None:
+            self.weight_log.append((w.data_ptr(), w.numel() * w.element_size()))
+        if self.prefetcher is not None:
+            self.prefetcher.after_product(self)
+
+    def _apply_stream_stages(self) -> None:
+        if self._stream_stages_set != self.STREAM_STAGES:
+            fn = _fn("gemm_stream", "iian_gemm_stream_stages", [c_int])
+            if fn(self.STREAM_STAGES) != 0:
+                raise KernelError("gemm_stream: the ring has 6 or 12 stages")
+            type(self)._stream_stages_set = self.STREAM_STAGES
 
     def linear_swiglu(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, row_scale=None) -> None:
         """out[t, f] = silu(x . w_gate_f) * (x . w_up_f) for w with gate and up rows interleaved in groups of 8."""
@@ -799,10 +844,14 @@ class CudaKernels:
 
     def attention_decode_fused(self, qkv, k_cache, v_cache, out, meta, *, num_heads, num_kv_heads, head_dim, scale, window,
                                q_weight, k_weight, eps, table, slots, write_kv: bool,
-                               n_split: Optional[int] = None, cluster: Optional[bool] = None) -> None:
+                               n_split: Optional[int] = None, cluster: Optional[bool] = None, sink: Optional[torch.Tensor] = None,
+                               softcap: Optional[float] = None, first_values: Optional[torch.Tensor] = None, share: float = 0.0) -> None:
         """Per-head RMSNorm, rotation, the write of the new K and V to the cache and attention over the cache in
         one launch, from the Q|K|V projection ``qkv`` [S, (nh + 2 nkv) * hd] of a step with one token per sequence.
-        Without ``write_kv`` the projection holds Q only ([S, nh * hd] is not accepted: pass the full width)."""
+        Without ``write_kv`` the projection holds Q only ([S, nh * hd] is not accepted: pass the full width).
+        ``sink``: float32 [heads], a logit per head in the denominator; ``softcap``: scores through ``c tanh(./c)``;
+        ``first_values`` (bf16 [S, nkv * hd], may be a column slice): what is stored and attended to is
+        ``(1 - share) v + share first_values``."""
         s_ = meta.num_seqs
         width = (num_heads + 2 * num_kv_heads) * head_dim
         if qkv.shape != (s_, width) or out.shape != (s_, num_heads * head_dim):
@@ -828,17 +877,23 @@ class CudaKernels:
             part_lse = part_o + rows * n_split * head_dim * 4
             counters = self.attention_counters(qkv.device, s_ * num_kv_heads).data_ptr()
         bt = meta.block_table
-        fn = _fn("attention_mma", "iian_attention_decode_fused",
+        fp, ld_f = self._rows(first_values, "first values")
+        if first_values is not None and (first_values.shape != (s_, num_kv_heads * head_dim) or first_values.dtype != qkv.dtype) \
+                or (sink is not None and sink.numel() != num_heads):
+            raise KernelError("attention_decode_fused: first values [S, nkv * hd], one sink per head")
+        fn = _fn("attention_mma", "iian_attention_decode_fused_mixed",
                  [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                   c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int,
-                  c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p])
+                  c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_float, c_void_p, c_longlong, c_float,
+                  c_float, c_void_p])
         _check(fn(_cuda(qkv, "qkv"), _cuda(k_cache, "k cache"), _cuda(v_cache, "v cache"), _cuda(out, "attention out"),
                   part_o, part_lse, counters, _cuda(meta.cu_q, "cu_q", torch.int32), _cuda(meta.ctx_len, "ctx_len", torch.int32),
                   _cuda(bt, "block table", torch.int32), bt.shape[1], s_, num_heads, num_kv_heads, head_dim,
                   k_cache.shape[2], k_cache.shape[0], scale, window or 0, n_split, 1 if cluster else 0,
                   _cuda(q_weight, "q norm weight", torch.float32), _cuda(k_weight, "k norm weight", torch.float32),
                   _cuda(table, "rotation table", torch.float32), _cuda(slots, "slots", torch.int32), eps,
-                  1 if write_kv else 0, self._decode_status(qkv.device), _stream()), "attention_decode_fused")
+                  1 if write_kv else 0, self._decode_status(qkv.device), _cuda(sink, "sink", torch.float32), softcap or 0.0, fp, ld_f,
+                  1.0 - share, share, _stream()), "attention_decode_fused")
 
     def paged_attention_generic(self, q, k_cache, v_cache, out, meta, *, num_heads, num_kv_heads, head_dim, scale,
                                 window) -> None:
@@ -909,11 +964,12 @@ class CudaKernels:
                   terms[0].shape[0], 1 if last_is_selected else 0, _cuda(out, "mix out", torch.float32), _cuda(out_act, "mix out"),
                   _code(out_act, "mix out") if out_act is not None else F32, r, h, _stream()), "depth_mix")
 
-    ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2, "relu2": 3}
+    ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2, "relu2": 3, "relu": 4}        # csrc/gated.cuh
 
     def gated_act(self, gate_up: torch.Tensor, out: torch.Tensor, interleave: int, activation: str, limit: float = 0.0) -> None:
         """``out = act(gate) * up`` for rows ``[gate | up]`` (or interleaved in groups of 8); ``gate_up`` may be a column slice.
-        ``clamped_swish`` (with ``limit``): ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``, ``g sigmoid(1.702 g) (u + 1)``."""
+        ``clamped_swish`` (with ``limit``): ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``, ``g sigmoid(1.702 g) (u + 1)``;
+        ``relu``: ``max(gate, 0) * up``."""
         n, f2 = gate_up.shape
         if out.shape != (n, f2 // 2) or f2 % 2 or out.dtype != gate_up.dtype:
             raise KernelError("gated_act: out must be [N, F] for gate_up [N, 2F] of the same dtype")
@@ -1089,16 +1145,15 @@ class CudaKernels:
 
     def moe_tcgen05_ok(self, dtype: torch.dtype, hidden: int, inter: int, activation: str) -> bool:
         """Whether both grouped products of an expert feed-forward can run on the tcgen05 kernel: bfloat16, rows of 16
-        bytes' multiples for TMA, gate and up interleaved in groups of 8 (SiLU, and the squared positive part of experts without
-        a gate, ride in the product's epilogue; the clamped activation is a pass of its own between the two products)."""
+        bytes' multiples for TMA, gate and up interleaved in groups of 8 (the activation rides in the first product's epilogue)."""
         return (self.MOE_TCGEN05 and not self.LIBRARY_GEMM_ONLY and dtype == torch.bfloat16
-                and activation in ("silu", "clamped_swish", "relu2") and hidden % 8 == 0 and inter % 8 == 0)
+                and activation in ("silu", "clamped_swish", "relu", "relu2") and hidden % 8 == 0 and inter % 8 == 0)
 
     def moe_grouped_gemm_tc(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: torch.Tensor, tiles: torch.Tensor,
-                            gated: bool, relu2: bool = False) -> None:
+                            gated: bool, relu2: bool = False, activation: str = "silu", limit: float = 0.0) -> None:
         """Rows of ``x`` sorted by expert times that expert's block of ``w`` [E, n, K] on tcgen05; ``gated``: the block's
-        rows are gate and up interleaved in groups of 8 and ``out`` [M, n / 2] = silu(gate) * up; ``relu2`` (not gated): ``out``
-        = max(product, 0)^2.  The plan's row tiles are of 128 rows."""
+        rows are gate and up interleaved in groups of 8 and ``out`` [M, n / 2] = act(gate, up) (``activation`` as in ``gated_act``);
+        ``relu2`` (not gated): ``out`` = max(product, 0)^2.  The plan's row tiles are of 128 rows."""
         m, k = x.shape
         e, n = w.shape[0], w.shape[1]
         if w.shape[2] != k or out.shape != (m, n // 2 if gated else n) or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 \
@@ -1108,10 +1163,11 @@ class CudaKernels:
         status = self.tcgen05_status_buffer(x.device).data_ptr()
         CudaKernels._tc_used = True
         fn = _fn("gemm_tcgen05", "iian_gemm_tcgen05_grouped",
-                 [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                  c_void_p])
-        _check(fn(_cuda(x, "moe rows"), _cuda(w, "expert weights"), _cuda(out, "moe out"), BF16, m, n, e, k, 1 if gated else 3 if relu2 else 0, bn,
-                  status, _cuda(tiles, "tiles", torch.int32), _cuda(offsets, "offsets", torch.int32), (tiles.numel() - 1) // 2,
+                 [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p,
+                  c_void_p, c_int, c_void_p])
+        epilogue = (1 if activation == "silu" else 4) if gated else 3 if relu2 else 0
+        _check(fn(_cuda(x, "moe rows"), _cuda(w, "expert weights"), _cuda(out, "moe out"), BF16, m, n, e, k, epilogue,
+                  self.ACTIVATIONS[activation], limit, bn, status, _cuda(tiles, "tiles", torch.int32), _cuda(offsets, "offsets", torch.int32), (tiles.numel() - 1) // 2,
                   _stream()), "gemm_tcgen05_grouped")
 
     def moe_route(self, logits: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.Tensor) -> None:
@@ -1176,6 +1232,26 @@ class CudaKernels:
         fn = _fn("elementwise", "iian_embedding_scaled", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p])
         _check(fn(_cuda(table, "embedding table"), _code(table, "embedding table"), _cuda(tokens, "tokens", torch.int32),
                   _cuda(out, "embedding out", torch.float32), n, h, table.shape[0], scale, _stream()), "embedding_scaled")
+
+    def embedding_placed(self, table: torch.Tensor, tokens: torch.Tensor, scale: float, places: Optional[torch.Tensor],
+                         positions: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, out: torch.Tensor,
+                         copy: Optional[torch.Tensor]) -> None:
+        """``out`` (float32) = ``table[token] * scale`` plus the row of ``places`` (same dtype as ``table``) for the token's position,
+        then divided by the row's root mean square and multiplied by ``weight``; ``copy`` receives it in its own dtype.  ``places``,
+        ``weight`` and ``copy`` may be None."""
+        n, h = out.shape
+        if table.shape[1] != h or tokens.numel() != n or (places is not None and (places.shape[1] != h or places.dtype != table.dtype
+                                                                                  or positions is None or positions.numel() != n)) \
+                or (weight is not None and weight.numel() != h) or (copy is not None and copy.shape != out.shape):
+            raise KernelError("embedding_placed: tables, weight and copy must fit the stream")
+        fn = _fn("residual_ops", "iian_embedding_placed",
+                 [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                  c_int, c_void_p])
+        _check(fn(_cuda(table, "embedding table"), _cuda(places, "position table"), _code(table, "embedding table"),
+                  _cuda(tokens, "tokens", torch.int32), _cuda(positions if places is not None else None, "positions", torch.int32), scale,
+                  _cuda(weight, "norm weight", torch.float32), eps, _cuda(out, "embedding out", torch.float32), _cuda(copy, "embedding copy"),
+                  _code(copy, "embedding copy") if copy is not None else F32, n, h, table.shape[0],
+                  places.shape[0] if places is not None else 0, _stream()), "embedding_placed")
 
     def add2_rms_norm(self, residual: torch.Tensor, delta: torch.Tensor, delta2: torch.Tensor, weight: torch.Tensor, eps: float,
                       out: torch.Tensor) -> None:
@@ -1485,16 +1561,27 @@ class CudaKernels:
         return {"n_split": self.attention_splits(num_seqs, num_kv_heads, min(max_ctx, chunk or window or max_ctx))}
 
     def _chunked_attention_mma(self, qp, ld_q, k_cache, v_cache, out, meta, nh, nkv, hd, scale, chunk, window, r1, r2, gp, ld_g,
-                               n, n_split, sink=None, keep_first: int = 0, gate_per_head: bool = False) -> None:
+                               n, n_split, sink=None, keep_first: int = 0, gate_per_head: bool = False,
+                               softcap: Optional[float] = None, score_bound: float = 0.0) -> None:
         if k_cache.shape[1] != nkv or k_cache.shape[3] != hd or v_cache.shape != k_cache.shape:
             raise KernelError("chunked_attention: cache shapes do not match the head counts")
         bt = meta.block_table
         if self.ATTENTION_TC and hd == 128 and k_cache.shape[2] in (8, 16, 32, 64, 128) and ld_q % 8 == 0 \
                 and meta.max_q_len * (nh // nkv) >= self.TC_ATTENTION_MIN_ROWS and (gate_per_head or (gp % 16 == 0 and ld_g % 8 == 0)) \
-                and out.data_ptr() % 16 == 0:
+                and out.data_ptr() % 16 == 0 and not (softcap and (gp or chunk or keep_first)):
             # portions of prompts with heads of 128: tcgen05 (csrc/attention_tc.cu)
             status = self.tcgen05_status_buffer(out.device)
             CudaKernels._tc_used = True
+            if softcap:
+                fn = _fn("attention_tc", "iian_attention_tc_capped",
+                         [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                          c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p])
+                _check(fn(qp, ld_q, _cuda(k_cache, "key cache"), _cuda(v_cache, "value cache"), _cuda(out, "attention out"),
+                          _cuda(meta.cu_q, "cu_q", torch.int32), _cuda(meta.ctx_len, "ctx_len", torch.int32),
+                          _cuda(bt, "block table", torch.int32), bt.shape[1], n, meta.num_seqs, meta.max_q_len, nh, nkv, hd,
+                          k_cache.shape[2], k_cache.shape[0], scale, window or 0, softcap, score_bound, status.data_ptr(),
+                          _cuda(sink, "sink", torch.float32), _stream()), "capped attention (tcgen05)")
+                return
             fn = _fn("attention_tc", "iian_attention_tc_kept",
                      [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                       c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -1522,17 +1609,18 @@ class CudaKernels:
             part_lse = part_o + rows * n_split * hd * 4
             row_tiles = -(-meta.max_q_len * (nh // nkv) // 16)
             counters = self.attention_counters(out.device, meta.num_seqs * nkv * row_tiles).data_ptr()
-        fn = _fn("attention_mma", "iian_attention_mma_kept",
+        fn = _fn("attention_mma", "iian_attention_mma_capped",
                  [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                   c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_void_p,
-                  c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p])
+                  c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_void_p])
         _check(fn(qp, ld_q, _cuda(k_cache, "key cache"), _cuda(v_cache, "value cache"), _cuda(out, "attention out"),
                   part_o, part_lse, counters, _cuda(meta.cu_q, "cu_q", torch.int32), _cuda(meta.ctx_len, "ctx_len", torch.int32),
                   _cuda(bt, "block table", torch.int32), bt.shape[1], n, meta.num_seqs, meta.max_q_len, nh, nkv, hd,
                   k_cache.shape[2], k_cache.shape[0], scale, window or 0, chunk or 0, n_split,
                   (2 if cluster else 1) if small else 0, self._decode_status(out.device) if small else None,
                   _cuda(sink, "sink", torch.float32), _cuda(r1, "r1", torch.float32), _cuda(r2, "r2", torch.float32), gp, ld_g,
-                  keep_first, 1 if gate_per_head else 0, _stream()), "chunked attention (mma)")
+                  keep_first, 1 if gate_per_head else 0, softcap or 0.0, _stream()),
+               "capped attention (mma)" if softcap else "chunked attention (mma)")
 
     # ---- a sub-layer output that passes a norm of its own before it joins the stream (csrc/residual_ops.cu) -----------------
     def normed_add_rms_norm(self, residual: torch.Tensor, y: Optional[torch.Tensor], post_weight: Optional[torch.Tensor],
@@ -1540,7 +1628,7 @@ class CudaKernels:
                             out: Optional[torch.Tensor]) -> None:
         """``residual += y / sqrt(mean(y^2) + post_eps) * post_weight`` (``y`` as it is without ``post_weight``) ``+ extra``
         (float32 rows), all in float32 and in place; ``out`` (optional) receives ``residual / sqrt(mean(residual^2) + eps) *
-        weight``.  Each of ``y``, ``extra``, ``out`` may be None."""
+        weight``; without ``weight`` the stream itself.  Each of ``y``, ``extra``, ``out`` may be None."""
         n, h = residual.shape
         act = out if out is not None else y
         if act is None:
@@ -1552,7 +1640,7 @@ class CudaKernels:
                 raise KernelError(f"normed_add_rms_norm: {name} {tuple(t.shape)} {t.dtype} does not match the stream {tuple(residual.shape)}")
         if extra is not None and (extra.shape != residual.shape or extra.dtype != torch.float32):
             raise KernelError("normed_add_rms_norm: the second addend must be float32 rows of the stream's shape")
-        if (out is not None and (weight is None or weight.numel() != h)) or (post_weight is not None and post_weight.numel() != h):
+        if (weight is not None and weight.numel() != h) or (post_weight is not None and post_weight.numel() != h):
             raise KernelError("normed_add_rms_norm: a norm's weight does not match the stream")
         fn = _fn("residual_ops", "iian_normed_add_rms_norm",
                  [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p])
@@ -1642,6 +1730,33 @@ class CudaKernels:
                   num_heads, num_kv_heads if k_cache is not None else 0, k_dim, v_dim, rot_dim, page, cells, eps, 1 if unit_norm else 0,
                   _stream()), "rotate_unit_store")
 
+    def head_norm_store(self, proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: torch.Tensor, k_cache: torch.Tensor,
+                        v_cache: torch.Tensor, slots: torch.Tensor, *, num_heads: int, num_kv_heads: int, k_dim: int, v_dim: int,
+                        q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
+                        first_values: Optional[torch.Tensor] = None, share: float = 0.0) -> None:
+        """Per token: every head of q and k divided by its root mean square, times a weight per entry (None: as projected); q to
+        ``q_out`` [N, heads, k_dim], k to its cache cells; the values, ``(1 - share) v + share first_values`` (``first_values`` [N,
+        nkv * v_dim], may be a column slice; None: as projected), to theirs."""
+        n = proj.shape[0]
+        pp, ld = self._rows(proj, "projections")
+        fp, ld_f = self._rows(first_values, "first values")
+        if q_out.shape != (n, num_heads, k_dim) or q_out.dtype != proj.dtype:
+            raise KernelError("head_norm_store: q_out must be [N, heads, k_dim] in the projections' dtype")
+        if k_cache.shape[1] != num_kv_heads or k_cache.shape[3] != k_dim or v_cache.shape[3] != v_dim \
+                or k_cache.shape[:3] != v_cache.shape[:3] or k_cache.dtype != proj.dtype or slots.numel() != n:
+            raise KernelError(f"head_norm_store: caches {tuple(k_cache.shape)} / {tuple(v_cache.shape)} do not fit")
+        if first_values is not None and (first_values.shape != (n, num_kv_heads * v_dim) or first_values.dtype != proj.dtype):
+            raise KernelError("head_norm_store: first values must be [N, nkv * v_dim] in the projections' dtype")
+        if any(w is not None and w.numel() != k_dim for w in (q_weight, k_weight)):
+            raise KernelError("head_norm_store: one weight per entry of a head")
+        fn = _fn("window_attention", "iian_head_norm_store",
+                 [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_float,
+                  c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_longlong, c_float, c_void_p])
+        _check(fn(pp, ld, q_off, k_off, v_off, _cuda(q_out, "queries"), _cuda(k_cache, "key cache"), _cuda(v_cache, "value cache"),
+                  _cuda(q_weight, "q norm weight", torch.float32), _cuda(k_weight, "k norm weight", torch.float32), fp, ld_f, 1.0 - share,
+                  share, _cuda(slots, "slots", torch.int32), _code(proj, "projections"), n, num_heads, num_kv_heads, k_dim, v_dim,
+                  k_cache.shape[2], k_cache.shape[0] * k_cache.shape[2], eps, _stream()), "head_norm_store")
+
     WINDOW_ATTENTION_MMA = os.environ.get("IIAN_WINDOW_ATTENTION_MMA", "1") not in ("0", "false", "off")
 
     def window_attention_mma_ok(self, dtype, num_heads: int, num_kv_heads: int, k_dim: int, v_dim: int, scale: float) -> bool:
@@ -1657,8 +1772,9 @@ class CudaKernels:
     def window_attention(self, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, meta, *,
                          num_heads: int, num_kv_heads: int, k_dim: int, v_dim: int, scale: float, window: Optional[int],
                          keep_first: int, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], gate_per_head: bool,
-                         n_split: Optional[int] = None) -> None:
-        """``q`` [N, heads * k_dim] -> ``out`` [N, heads * v_dim]: softmax of ``q . k * scale`` over the keys ``j <= i`` with
+                         n_split: Optional[int] = None, softcap: Optional[float] = None, score_bound: float = 0.0) -> None:
+        """``q`` [N, heads * k_dim] -> ``out`` [N, heads * v_dim]: softmax of ``q . k * scale`` (through ``c tanh(./c)`` with
+        ``softcap`` c; ``score_bound``: a number no score exceeds before the cap, 0: not known) over the keys ``j <= i`` with
         ``i - j < window`` or ``j < keep_first``, the denominator also holding ``exp(sink_h)`` if given; weighted sum of the
         cached values, times ``sigmoid(gate)``: one number per head (``gate_per_head``: rows of ``heads`` numbers) or per entry
         (rows of ``heads * v_dim``); the gate may be a column slice.  In bfloat16 with keys and values of 64 or 128 entries
@@ -1675,16 +1791,16 @@ class CudaKernels:
                 and qp % 16 == 0 and (gate is None or gate_per_head or (ld_g % 2 == 0 and gp % 4 == 0)):
             self._chunked_attention_mma(qp, ld_q, k_cache, v_cache, out, meta, num_heads, num_kv_heads, k_dim, scale, None, window,
                                         None, None, gp, ld_g, n, n_split, sink=sink, keep_first=keep_first if window else 0,
-                                        gate_per_head=gate is not None and gate_per_head)
+                                        gate_per_head=gate is not None and gate_per_head, softcap=softcap, score_bound=score_bound)
             return
         bt = meta.block_table
         fn = _fn("window_attention", "iian_window_attention",
                  [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
-                  c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p])
+                  c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p])
         _check(fn(qp, ld_q, _cuda(k_cache, "key cache"), _cuda(v_cache, "value cache"), _cuda(out, "attention out"),
                   _cuda(meta.positions, "positions", torch.int32), _cuda(meta.seq_of_token, "seq_of_token", torch.int32),
                   _cuda(bt, "block table", torch.int32), bt.shape[1], _cuda(meta.ctx_len, "ctx_len", torch.int32), _code(q, "queries"),
-                  n, num_heads, num_kv_heads, k_dim, v_dim, k_cache.shape[2], k_cache.shape[0], scale, window or 0, keep_first,
+                  n, num_heads, num_kv_heads, k_dim, v_dim, k_cache.shape[2], k_cache.shape[0], scale, softcap or 0.0, window or 0, keep_first,
                   _cuda(sink, "sink", torch.float32), gp, ld_g, 1 if gate_per_head else 0, _stream()), "window_attention")
 
     # ---- heads as the difference of two softmax maps over the same values (csrc/difference_attention.cu) ------------------------

@@ -16,10 +16,10 @@ Two further forms, chosen by parameters.  ``score = "table"``: there is no route
 "clamped_swish"``: ``g = min(Wgate u, limit)``, ``v = clamp(Wup u, -limit, limit)``, the expert's hidden row is
 ``g sigmoid(1.702 g) (v + 1)``.
 
-``score = "softmax_top"``: the router has a bias (``router.b``, float32 sum), the ``top`` experts with the largest biased
+``score = "softmax_top"``: the router has a bias (``router.b``, float32 sum) unless ``router_bias`` is false, the ``top`` experts with the largest biased
 logits are taken and weighed by the softmax over those logits ALONE.  ``shared_intermediate_size``: one more gated
-feed-forward of that width (tensors ``shared.gate / up / down``, same activation) that every token uses; its output is added
-to the experts' sum in the kernel that forms it.
+feed-forward of that width (tensors ``shared.gate / up / down``, same activation, ``shared_limit`` for the clamped one) that every
+token uses; its output is added to the experts' sum in the kernel that forms it.
 
 ``score = "softmax"``: scores are the softmax over all router outputs, without a bias; the ``top`` outputs with the largest
 score plus ``correction`` (a number per output that only the choice sees) are taken and weighed by ``weight_scale`` times their
@@ -46,9 +46,9 @@ from .base import FeedForward, register_feed_forward
 @register_feed_forward("routed_experts")
 class RoutedExperts(FeedForward):
     """params: ``hidden_size``, ``num_experts``, ``top``, ``intermediate_size`` (of one expert), ``activation``
-    (``silu`` | ``gelu_tanh`` | ``clamped_swish`` with ``limit`` | ``relu2``), ``score`` (``sigmoid`` | ``softmax_top`` | ``softmax``
-    with ``weight_scale`` and ``identity_experts`` | ``table`` with ``vocab_size``), ``weight_on`` (``input`` | ``output``),
-    ``shared_intermediate_size`` with ``shared_gate``."""
+    (``silu`` | ``gelu_tanh`` | ``clamped_swish`` with ``limit`` | ``relu2``), ``score`` (``sigmoid`` | ``softmax_top`` with
+    ``router_bias`` | ``softmax`` with ``weight_scale`` and ``identity_experts`` | ``table`` with ``vocab_size``), ``weight_on`` (``input`` | ``output``),
+    ``shared_intermediate_size`` with ``shared_gate`` and ``shared_limit``."""
 
     SWISH_ALPHA = 1.702         # fixed by the clamped activation (also in the kernels)
 
@@ -80,8 +80,6 @@ class RoutedExperts(FeedForward):
         self.shared_inter = int(p.get("shared_intermediate_size", 0) or 0)
         self.shared = None
         if self.shared_inter:
-            if self.activation not in ("silu", "gelu_tanh", "relu2"):
-                raise ValueError("routed_experts: the shared expert takes silu, gelu_tanh or relu2")
             from ..config.spec import PartSpec
             from .mlp import GatedMLP, PlainMLP
             if self.activation == "relu2":
@@ -91,10 +89,12 @@ class RoutedExperts(FeedForward):
             else:
                 self.shared = GatedMLP(PartSpec("gated_mlp", {"hidden_size": self.hidden, "intermediate_size": self.shared_inter,
                                                               "activation": self.activation,
+                                                              "limit": float(p.get("shared_limit", self.limit)),
                                                               "names": ("shared.gate", "shared.up", "shared.down")}), dtype, device)
         self.shared_gate = bool(p.get("shared_gate", False)) and self.shared is not None
-        if self.shared_gate and self.score != "softmax":
-            raise ValueError("routed_experts: shared_gate comes with score 'softmax'")
+        if self.shared_gate and self.score not in ("softmax", "softmax_top"):
+            raise ValueError("routed_experts: shared_gate comes with score 'softmax' or 'softmax_top'")
+        self.has_router_bias = self.score == "softmax_top" and bool(p.get("router_bias", True))
         self.router_bias = None
         self.vocab = int(p["vocab_size"]) if self.score == "table" else 0
         self.needs_tokens = self.score == "table"       # forward wants to know which token each row belongs to
@@ -113,7 +113,7 @@ class RoutedExperts(FeedForward):
                 t["correction"] = TensorSpec((self.outputs,), init="zeros_jitter")
             if self.shared_gate:
                 t["shared.sg"] = TensorSpec((1, self.hidden))
-            if self.score == "softmax_top":
+            if self.has_router_bias:
                 t["router.b"] = TensorSpec((self.experts,))
         if self.shared is not None:
             t.update(self.shared.tensors())
@@ -130,7 +130,7 @@ class RoutedExperts(FeedForward):
         else:
             self._router = tensors["router"]
             self.w_router = self._router.contiguous()
-            if self.score == "softmax_top":
+            if self.has_router_bias:
                 self.router_bias = tensors["router.b"].to(torch.float32).contiguous()
             if self.score == "softmax":
                 self.correction = tensors["correction"].to(torch.float32).contiguous()
@@ -165,8 +165,6 @@ class RoutedExperts(FeedForward):
     def kernel_libraries(self):
         if self.shared is not None:
             return tuple(set(("moe", "gemm_simt") + tuple(self.shared.kernel_libraries())))
-        if self.activation == "clamped_swish" and self.dtype == torch.bfloat16:
-            return ("moe", "gemm_simt", "postnorm")      # the activation between the two tcgen05 products
         return ("moe", "gemm_simt")        # in bfloat16 the products' fast forms come with gemm_simt (the grouped tcgen05 one too)
 
     def forward(self, x, ctx, with_extra: bool = False, rows=None):
@@ -213,13 +211,8 @@ class RoutedExperts(FeedForward):
             else:
                 k.moe_grouped_gemm(xs, self.w_up, None, act, offsets, tiles, "relu2")
                 k.moe_grouped_gemm(act, self.w_down, None, ys, offsets, tiles)
-        elif on_tc and self.activation != "silu":
-            wide = ctx.buf("expert_gate_up", (m, 2 * self.inter), self.dtype)
-            k.moe_grouped_gemm_tc(xs, self.w_gate_up, wide, offsets, tiles, gated=False)
-            k.gated_act(wide, act, 8, self.activation, self.limit)
-            k.moe_grouped_gemm_tc(act, self.w_down, ys, offsets, tiles, gated=False)
         elif on_tc:
-            k.moe_grouped_gemm_tc(xs, self.w_gate_up, act, offsets, tiles, gated=True)
+            k.moe_grouped_gemm_tc(xs, self.w_gate_up, act, offsets, tiles, gated=True, activation=self.activation, limit=self.limit)
             k.moe_grouped_gemm_tc(act, self.w_down, ys, offsets, tiles, gated=False)
         else:
             if self.w_gate_up is not None:
@@ -227,7 +220,7 @@ class RoutedExperts(FeedForward):
             else:
                 k.moe_grouped_gemm(xs, self.w_gate, self.w_up, act, offsets, tiles, self.activation, self.limit)
             k.moe_grouped_gemm(act, self.w_down, None, ys, offsets, tiles)
-        if self.score == "softmax":
+        if self.score == "softmax" or self.shared_gate:
             add = self.shared.forward(x, ctx) if self.shared is not None else None        # lands in "ffn_out" and is summed in place
             out = add if add is not None else ctx.buf("ffn_out", (n, self.hidden), self.dtype)
             k.moe_combine_mixed(ys, pos, wts, x, out, top, add, logits[:, self.outputs: self.outputs + 1] if self.shared_gate else None)

@@ -7,7 +7,8 @@ Gate and up projections run as one matrix product over the rows of both, stacked
 consecutive rows holds both halves of 8 features and can apply SiLU(gate) * up in its epilogue.  If the
 intermediate size is no multiple of 8 the rows are stacked as ``Wgate | Wup``.
 
-``activation``: ``silu`` or ``gelu_tanh`` (``0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))``); the second has no
+``activation``: ``silu``, ``relu`` (``max(z, 0)``), ``clamped_swish`` (with ``limit``: ``g = min(gate, limit)``, ``u = clamp(up, -limit,
+limit)``, ``g sigmoid(1.702 g) (u + 1)``) or ``gelu_tanh`` (``0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))``); the last has no
 fused product epilogue and runs as product, then activation kernel.  ``stack_rows`` puts further rows that read the same
 input (a gate of the residual) under ``Wgate | Wup`` so that one product serves all.
 """
@@ -24,7 +25,8 @@ from .base import FeedForward, Prenormed, register_feed_forward
 
 @register_feed_forward("gated_mlp")
 class GatedMLP(FeedForward):
-    """params: ``hidden_size``, ``intermediate_size``, ``activation`` (``silu`` | ``gelu_tanh``); optional ``names``: the
+    """params: ``hidden_size``, ``intermediate_size``, ``activation`` (``silu`` | ``gelu_tanh`` | ``relu`` | ``clamped_swish`` with
+    ``limit``); optional ``names``: the
     local tensor names of (gate, up, down)."""
 
     def __init__(self, spec, dtype, device):
@@ -32,9 +34,12 @@ class GatedMLP(FeedForward):
         self.hidden = int(spec["hidden_size"])
         self.inter = int(spec["intermediate_size"])
         act = spec.params.get("activation", "silu")
-        if act not in ("silu", "gelu_tanh"):
-            raise ValueError(f"gated_mlp: activation '{act}' has no kernel (silu, gelu_tanh)")
+        if act not in ("silu", "gelu_tanh", "relu", "clamped_swish"):
+            raise ValueError(f"gated_mlp: activation '{act}' has no kernel (silu, gelu_tanh, relu, clamped_swish)")
         self.activation = act
+        self.limit = float(spec.params.get("limit", 0.0))
+        if act == "clamped_swish" and self.limit <= 0:
+            raise ValueError("gated_mlp: the clamped activation needs a positive limit")
         self.names = tuple(spec.params.get("names", ("gate_proj.weight", "up_proj.weight", "down_proj.weight")))
         self.w_gate_up = self.w_down = None
         self.interleave = 0
@@ -89,7 +94,7 @@ class GatedMLP(FeedForward):
         wide = ctx.buf("gate_up", (n, w.shape[0]), self.dtype)
         k.linear(x, w, wide)
         act = ctx.buf("ffn_act", (n, self.inter), self.dtype)
-        k.gated_act(wide[:, : 2 * self.inter], act, self.interleave, self.activation)
+        k.gated_act(wide[:, : 2 * self.inter], act, self.interleave, self.activation, self.limit)
         out = ctx.buf("ffn_out", (n, self.hidden), self.dtype)
         k.linear(act, self.w_down, out)
         if with_extra:
@@ -97,9 +102,17 @@ class GatedMLP(FeedForward):
         return out
 
     def forward(self, x, ctx, norm_out=None, with_extra: bool = False):
-        if with_extra or self.activation != "silu":
-            return self._forward_general(x, ctx, with_extra)
         k = ops.kernels()
+        if with_extra:
+            return self._forward_general(x, ctx, with_extra)
+        if self.activation != "silu":
+            if not (hasattr(k, "can_fuse_gated") and k.can_fuse_gated(x, self.w_gate_up, self.interleave, self.activation)):
+                return self._forward_general(x, ctx, with_extra)
+            act = ctx.buf("ffn_act", (x.shape[0], self.inter), self.dtype)
+            k.linear_gated(x, self.w_gate_up, act, self.activation, self.limit)
+            out = ctx.buf("ffn_out", (x.shape[0], self.hidden), self.dtype)
+            k.linear(act, self.w_down, out)
+            return out
         scale = None
         if isinstance(x, Prenormed):
             x, scale = x.x, x.scale

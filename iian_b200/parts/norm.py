@@ -76,6 +76,38 @@ class RMSNorm(Norm):
         return out
 
 
+@register_norm("identity")
+class Identity(Norm):
+    """No norm in a norm's place: the sub-layer behind it reads the stream itself.  No params, no tensors.
+
+    What is still owed to the stream (a tensor or a ``NormedAddend``) is added first, as every norm does, and the stream's copy in
+    the activation dtype leaves the same kernel.  Whoever wrote the stream last may have left that copy already
+    (``ctx.step_cache["stream_act"]``); in 32-bit the stream is its own copy."""
+
+    def kernel_libraries(self):
+        return ("residual_ops",)
+
+    def forward(self, residual: torch.Tensor, delta, ctx, delta_scale: float = 1.0) -> torch.Tensor:
+        if delta_scale != 1.0 or isinstance(delta, tuple):
+            raise ValueError("identity: one addend, without a factor")
+        if delta is not None and not isinstance(delta, NormedAddend):
+            delta = NormedAddend(delta, None, 0.0)
+        k = ops.kernels()
+        copy = ctx.step_cache.pop("stream_act", None)
+        if self.dtype == torch.float32:
+            if delta is not None:
+                k.normed_add_rms_norm(residual, delta.y, delta.weight, delta.eps, delta.extra, None, 0.0, None)
+            return residual
+        if delta is None and copy is not None and copy.shape == residual.shape:
+            return copy
+        out = ctx.buf("normed", residual.shape, self.dtype)
+        if delta is None:
+            k.normed_add_rms_norm(residual, None, None, 0.0, None, None, 0.0, out)
+        else:
+            k.normed_add_rms_norm(residual, delta.y, delta.weight, delta.eps, delta.extra, None, 0.0, out)
+        return out
+
+
 @register_norm("layer_norm")
 class LayerNorm(Norm):
     """params: ``size``, ``eps``.  ``y = (x - mean) / sqrt(var + eps) * w + b`` with ``var`` the mean of the squared

@@ -278,14 +278,20 @@ class FakeKernels:
             return z / (1 + torch.exp(-z))
         return 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
 
-    def gated_act(self, gate_up, out, interleave, activation):
+    def gated_act(self, gate_up, out, interleave, activation, limit=0.0):
         f = out.shape[1]
         if interleave:
             v = gate_up.float().reshape(gate_up.shape[0], f // 8, 2, 8)
             g, u = v[:, :, 0].reshape(-1, f), v[:, :, 1].reshape(-1, f)
         else:
             g, u = gate_up[:, :f].float(), gate_up[:, f:].float()
-        out.copy_((self._act(g, activation) * u).to(out.dtype))
+        if activation == "clamped_swish":
+            g, u = g.clamp(max=limit), u.clamp(-limit, limit) + 1
+            out.copy_((g * torch.sigmoid(1.702 * g) * u).to(out.dtype))
+        elif activation == "relu":
+            out.copy_((torch.relu(g) * u).to(out.dtype))
+        else:
+            out.copy_((self._act(g, activation) * u).to(out.dtype))
 
     # ---- attention over a cached latent ------------------------------------------------------------------
     def latent_prep(self, qd, q_off, dkv_off, cache_rows, q_cat, norm_weight, inv_freq, positions, slots, *, num_heads, dim,
@@ -439,9 +445,21 @@ class FakeKernels:
             residual.add_(v)
         if extra is not None:
             residual.add_(extra)
-        if out is not None:
+        if out is not None and weight is None:
+            out.copy_(residual.to(out.dtype))
+        elif out is not None:
             x = residual
             out.copy_((x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * weight).to(out.dtype))
+
+    def embedding_placed(self, table, tokens, scale, places, positions, weight, eps, out, copy):
+        x = table[tokens.long()].float() * scale
+        if places is not None:
+            x = x + places[positions.long().clamp(0, places.shape[0] - 1)].float()
+        if weight is not None:
+            x = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * weight
+        out.copy_(x)
+        if copy is not None:
+            copy.copy_(x.to(copy.dtype))
 
     def weighted_sum2(self, x, a, y, b, out):
         out.copy_((a * x.float() + b * y.float()).to(out.dtype))
@@ -490,8 +508,30 @@ class FakeKernels:
             k_cache[s // ps, :, s % ps, :] = k[t].to(k_cache.dtype)
             v_cache[s // ps, :, s % ps, :] = v[t].to(v_cache.dtype)
 
+    def head_norm_store(self, proj, q_off, k_off, v_off, q_out, k_cache, v_cache, slots, *, num_heads, num_kv_heads, k_dim, v_dim,
+                        q_weight, k_weight, eps, first_values=None, share=0.0):
+        n = proj.shape[0]
+
+        def norm(t, w):
+            t = t.float()
+            return t if w is None else t * torch.rsqrt((t * t).mean(-1, keepdim=True) + eps) * w
+
+        q_out.copy_(norm(proj[:, q_off:q_off + num_heads * k_dim].reshape(n, num_heads, k_dim), q_weight).to(q_out.dtype))
+        k = norm(proj[:, k_off:k_off + num_kv_heads * k_dim].reshape(n, num_kv_heads, k_dim), k_weight)
+        v = proj[:, v_off:v_off + num_kv_heads * v_dim].float()
+        if first_values is not None:
+            v = (1.0 - share) * v + share * first_values.float()
+        v = v.reshape(n, num_kv_heads, v_dim)
+        ps = k_cache.shape[2]
+        for t in range(n):
+            s = int(slots[t])
+            if s < 0:
+                continue
+            k_cache[s // ps, :, s % ps, :] = k[t].to(k_cache.dtype)
+            v_cache[s // ps, :, s % ps, :] = v[t].to(v_cache.dtype)
+
     def window_attention(self, q, k_cache, v_cache, out, meta, *, num_heads, num_kv_heads, k_dim, v_dim, scale, window, keep_first,
-                         sink, gate, gate_per_head, n_split=None):
+                         sink, gate, gate_per_head, n_split=None, softcap=None, score_bound=0.0):
         n = q.shape[0]
         ps = k_cache.shape[2]
         rep = num_heads // num_kv_heads
@@ -510,6 +550,9 @@ class FakeKernels:
             vv = v_cache[pages, :, (js % ps).long(), :].float()
             for h in range(num_heads):
                 sc = (kk[:, h // rep, :] @ qf[t, h]) * scale
+                if softcap:
+                    assert not score_bound or float(sc.abs().max()) <= score_bound, "a score beyond its bound"
+                    sc = softcap * torch.tanh(sc / softcap)
                 if sink is not None:
                     sc = torch.cat([sc, sink[h:h + 1]])
                 o[t, h] = torch.softmax(sc, dim=0)[: js.numel()] @ vv[:, h // rep, :]
