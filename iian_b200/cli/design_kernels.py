@@ -739,6 +739,170 @@ def run_ferodra(peaks: dict, width: int = 2048, heads: int = 16) -> dict:
     return out
 
 
+def run_tatelorn(peaks: dict, width: int = 2048, heads: int = 16) -> dict:
+    """The kernels of the Tatelorn design alone, each beside its like kernel at equal size (16 heads of 128 on 8 KV heads):
+      decode attention    8 (and 64) sequences of 4,096 cached tokens, one kernel from the projections on: norms, mixed values, cache
+                          write, capped scores, sink  vs  Qwen3's (norms, rotation, cache write)
+      prefill attention   one sequence of 2,048 tokens, and of 8,192: scores known to stay within half the cap, within the cap, not
+                          known  vs  Qwen3's
+      heads + cache       2,048 tokens: norms, mixed values, cache write  vs  Qwen3's norms, rotation, cache write
+      sum                 2,048 rows: a normalised addend and the stream's copy  vs  Nogelorn's with the next norm
+      stream's start      2,048 tokens: token row, position row, norm, copy  vs  the plain embedding
+      dense feed-forward  2,048 (and 8) rows: relu gate  vs  Qwen3's silu gate
+      expert products     2,048 (and 8) tokens x 5 of 64 clamped experts + a shared one with a sigmoid  vs  Nogelorn's with silu
+    """
+    import torch
+    from .. import ops
+    from ..config.spec import PartSpec
+    from ..engine.runner import StepContext, Workspace
+    from ..parts.experts import RoutedExperts
+    k = ops.kernels()
+    dev = torch.device("cuda:0")
+    bf = torch.bfloat16
+    nkv, hd, page, cap, scale = 8, 128, 16, 30.0, 128 ** -0.5
+    out = {}
+    hbm, tfl = peaks["hbm_gbs"], peaks["bf16_tflops"]
+
+    def mem_row(name, ms, nbytes):
+        out[name] = {"ms": ms, "gb_s": nbytes / ms / 1e6, "of_hbm_peak": nbytes / ms / 1e6 / hbm}
+
+    def flop_row(name, ms, flops):
+        out[name] = {"ms": ms, "tflops": flops / ms / 1e9, "of_bf16_peak": flops / ms / 1e9 / tfl}
+
+    sink = torch.zeros(heads, device=dev)
+    qw = torch.ones(hd, device=dev)
+    wide = (heads + 2 * nkv) * hd
+    inv64 = torch.pow(torch.tensor(500000.0, dtype=torch.float64), -torch.arange(hd // 2, dtype=torch.float64) / (hd // 2)).to(dev)
+    # ---- decode attention ---------------------------------------------------------------------------------------------------
+    for B, ctx in ((8, 4096), (64, 4096)):
+        meta, pages = _meta([ctx] * B, [1] * B, page, dev)
+        slots = torch.tensor([(s + 1) * ctx - 1 for s in range(B)], dtype=torch.int32, device=dev)
+        copies = [(torch.randn(pages, nkv, page, hd, device=dev).to(bf), torch.randn(pages, nkv, page, hd, device=dev).to(bf) * 0.3)
+                  for _ in range(2)]
+        proj = torch.randn(B, wide, device=dev).to(bf)
+        first = torch.randn(B, nkv * hd, device=dev).to(bf)
+        table = torch.empty(B, hd // 2, 2, device=dev)
+        k.rotary_table_scaled(inv64, meta.positions, hd // 2, 1.0, table)
+        o = torch.empty(B, heads * hd, device=dev, dtype=bf)
+        kw = dict(num_heads=heads, num_kv_heads=nkv, head_dim=hd, scale=scale, window=None, q_weight=qw, k_weight=qw, eps=1e-6, slots=slots,
+                  write_kv=True)
+        nbytes = B * ctx * 2 * nkv * hd * 2
+        ms = _timed([(lambda c=c: k.attention_decode_fused(proj, c[0], c[1], o, meta, table=None, sink=sink, softcap=cap, first_values=first,
+                                                           share=0.4, **kw)) for c in copies])
+        mem_row(f"decode_attention_capped_{B}x{ctx}", ms, nbytes)
+        ms = _timed([(lambda c=c: k.attention_decode_fused(proj, c[0], c[1], o, meta, table=table, **kw)) for c in copies])
+        mem_row(f"decode_attention_qwen3_{B}x{ctx}", ms, nbytes)
+        del copies
+    torch.cuda.empty_cache()
+    # ---- prefill attention ---------------------------------------------------------------------------------------------------
+    for T in (2048, 8192):
+        meta, pages = _meta([T], [T], page, dev)
+        kc = torch.randn(pages, nkv, page, hd, device=dev).to(bf)
+        vc = torch.randn(pages, nkv, page, hd, device=dev).to(bf) * 0.3
+        q = torch.randn(T, heads * hd, device=dev).to(bf)
+        o = torch.empty(T, heads * hd, device=dev, dtype=bf)
+        pairs = T * (T + 1) / 2
+        att = dict(num_heads=heads, num_kv_heads=nkv, k_dim=hd, v_dim=hd, scale=scale, window=None, keep_first=0, sink=sink, gate=None,
+                   gate_per_head=True)
+        for tag, kw in (("half_the_cap", {"softcap": cap, "score_bound": 0.5 * cap}), ("within_the_cap", {"softcap": cap, "score_bound": cap}),
+                        ("bound_not_known", {"softcap": cap}), ("not_known_beyond_the_cap", {"softcap": cap, "scale": 2.5}), ("no_cap", {})):
+            ms = _timed([lambda: k.window_attention(q, kc, vc, o, meta, **dict(att, **kw))] * 3)
+            flop_row(f"prefill_attention_{tag}_{T}", ms, 4.0 * heads * hd * pairs)
+        q3 = q.view(T, heads, hd)
+        ms = _timed([lambda: k.paged_attention(q3, kc, vc, o, meta, num_heads=heads, num_kv_heads=nkv, head_dim=hd, scale=scale,
+                                               window=None)] * 3)
+        flop_row(f"prefill_attention_qwen3_{T}", ms, 4.0 * heads * hd * pairs)
+        del kc, vc
+    torch.cuda.empty_cache()
+    # ---- norms of the heads, mixed values, cache write ---------------------------------------------------------------------------
+    T = 2048
+    meta, pages = _meta([T], [T], page, dev)
+    slots = torch.arange(T, dtype=torch.int32, device=dev)
+    sets = [(torch.randn(T, wide, device=dev).to(bf), torch.empty(T, heads, hd, device=dev, dtype=bf),
+             torch.zeros(pages, nkv, page, hd, device=dev, dtype=bf), torch.zeros(pages, nkv, page, hd, device=dev, dtype=bf),
+             torch.randn(T, wide, device=dev).to(bf)) for _ in range(4)]
+    ms = _timed([(lambda t=t: k.head_norm_store(t[0], 0, heads * hd, (heads + nkv) * hd, t[1], t[2], t[3], slots, num_heads=heads,
+                                                num_kv_heads=nkv, k_dim=hd, v_dim=hd, q_weight=qw, k_weight=qw, eps=1e-6,
+                                                first_values=t[4][:, (heads + nkv) * hd:], share=0.4)) for t in sets])
+    mem_row("head_norm_store", ms, (2 * T * wide + T * nkv * hd) * 2)
+    table = torch.empty(T, hd // 2, 2, device=dev)
+    k.rotary_table_scaled(inv64, meta.positions, hd // 2, 1.0, table)
+    inv32 = inv64.float()
+    ms = _timed([(lambda t=t: k.qk_norm_rope_store(t[0], t[1], t[2], t[3], num_heads=heads, num_kv_heads=nkv, head_dim=hd, q_weight=qw,
+                                                   k_weight=qw, eps=1e-6, inv_freq=inv32, rot_dim=hd, rope_style=0,
+                                                   positions=meta.positions, slots=slots, write_kv=True, table=table)) for t in sets])
+    mem_row("qk_norm_rope_store_qwen3", ms, 2 * T * wide * 2)
+    del sets
+    # ---- sums, the stream's start ----------------------------------------------------------------------------------------------------
+    w = torch.ones(width, device=dev)
+    for n in (2048, 8):
+        sets = [(torch.randn(n, width, device=dev), torch.randn(n, width, device=dev).to(bf), torch.empty(n, width, device=dev, dtype=bf))
+                for _ in range(8)]
+        ms = _timed([(lambda t=t: k.normed_add_rms_norm(t[0], t[1], w, 1e-6, None, None, 0.0, t[2])) for t in sets])
+        mem_row(f"normed_add_copy_{n}", ms, n * width * (4 + 2 + 4 + 2))
+        ms = _timed([(lambda t=t: k.normed_add_rms_norm(t[0], t[1], w, 1e-6, None, w, 1e-6, t[2])) for t in sets])
+        mem_row(f"normed_add_rms_norm_nogelorn_{n}", ms, n * width * (4 + 2 + 4 + 2))
+        emb, places = torch.randn(32768, width, device=dev).to(bf), torch.randn(8192, width, device=dev).to(bf)
+        ids = [torch.randint(0, 32768, (n,), dtype=torch.int32, device=dev) for _ in sets]
+        pos = [torch.randint(0, 8192, (n,), dtype=torch.int32, device=dev) for _ in sets]
+        ms = _timed([(lambda t=t, i=i, p=p: k.embedding_placed(emb, i, 45.0, places, p, w, 1e-6, t[0], t[2])) for t, i, p in zip(sets, ids, pos)])
+        mem_row(f"embedding_placed_{n}", ms, n * width * (2 + 2 + 4 + 2))
+        ms = _timed([(lambda t=t, i=i: k.embedding_scaled(emb, i, 45.0, t[0])) for t, i in zip(sets, ids)])
+        mem_row(f"embedding_scaled_nogelorn_{n}", ms, n * width * (2 + 4))
+        del sets, emb, places
+    # ---- dense feed-forward -----------------------------------------------------------------------------------------------------------
+    inter = 4 * width
+    for n in (2048, 8):
+        h = torch.randn(n, width, device=dev).to(bf)
+        ws = [(torch.randn(2 * inter, width, device=dev).to(bf) * 0.02, torch.randn(width, inter, device=dev).to(bf) * 0.02)
+              for _ in range(3 if n < 128 else 1)]
+        a2, y2 = torch.empty(n, inter, device=dev, dtype=bf), torch.empty(n, width, device=dev, dtype=bf)
+        gu = torch.empty(n, 2 * inter, device=dev, dtype=bf)
+
+        def dense_on(wa, wb, act):
+            def run_():
+                if act == "relu" and k.can_fuse_gated(h, wa, 8, act):
+                    k.linear_gated(h, wa, a2, act)
+                elif act == "silu" and k.can_fuse_swiglu(h, wa, 8):
+                    k.linear_swiglu(h, wa, a2)
+                else:
+                    k.linear(h, wa, gu)
+                    k.gated_act(gu, a2, 8, act) if act == "relu" else k.swiglu(gu, a2, 8)
+                k.linear(a2, wb, y2)
+            return run_
+        for act, tag in (("relu", "relu_feed_forward"), ("silu", "swiglu_feed_forward_qwen3")):
+            ms = _timed([dense_on(a, b, act) for a, b in ws] * (1 if n < 128 else 3))
+            if n >= 128:
+                flop_row(f"{tag}_{n}", ms, 2.0 * n * 3 * inter * width)
+            else:
+                mem_row(f"{tag}_{n}", ms, 3 * inter * width * 2)
+        del ws
+    # ---- expert products ---------------------------------------------------------------------------------------------------------------
+    E, ff, top = 64, 1408, 5
+    parts = {}
+    for name, params in (("clamped", {"activation": "clamped_swish", "limit": 7.0, "router_bias": False, "shared_gate": True, "shared_limit": 7.0}),
+                         ("softmax_nogelorn", {"activation": "silu"})):
+        part = RoutedExperts(PartSpec("routed_experts", dict(params, hidden_size=width, num_experts=E, top=top, weight_on="output",
+                                                             score="softmax_top", intermediate_size=ff, shared_intermediate_size=ff)), bf, dev)
+        part.bind({tn: torch.randn(*ts.shape, device=dev).to(bf) * (1.0 if tn.startswith("router") else 0.02) for tn, ts in part.tensors().items()})
+        parts[name] = part
+    for n in (2048, 64, 8, 1):
+        h = torch.randn(n, width, device=dev).to(bf)
+        for name, part in parts.items():
+            ctx_ = StepContext(Workspace(dev))
+            part.forward(h, ctx_)
+            ms = _timed(lambda: part.forward(h, ctx_))
+            ids = ctx_.buf("expert_ids", (n, top), torch.int32).flatten().tolist()
+            if n >= 128:
+                flop_row(f"expert_feed_forward_{name}_{n}", ms, 2.0 * (len(ids) + n) * 3 * ff * width)
+            else:
+                mem_row(f"expert_feed_forward_{name}_{n}", ms, (len(set(ids)) + 1) * 3 * ff * width * 2)
+    del parts
+    torch.cuda.empty_cache()
+    k.check_device_status()
+    return out
+
+
 def run_senadra(peaks: dict, width: int = 2048, heads: int = 16) -> dict:
     """The kernels of the Senadra design alone, each beside its like kernel of another path at equal size (16 heads of 128 on
     8 KV heads, chunks of 2,048 positions; recurrences of 16 value heads 128 x 128 on 8 query/key heads; latents of 512 + 64):

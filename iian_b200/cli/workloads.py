@@ -181,11 +181,49 @@ FERODRA_SHAPES: Dict[str, dict] = {
 }
 EQUAL_NOGELORN = {"f2k-moe": "n2k-moe", "f4k-moe": "n4k-moe"}
 EQUAL_QWEN3.update({f: EQUAL_QWEN3[n] for f, n in EQUAL_NOGELORN.items()})
+
+
+def _tatelorn_shape(width, heads, experts, top, expert_ff, vocab=32768, positions=16384):
+    """Eight attention layers: normed heads of 128 on 8 key/value heads, scores through a cap of 30, values mixed with the first
+    layer's; a dense relu feed-forward as wide as the active experts in the first layer, clamped experts with one more that every
+    token uses behind the others."""
+    att = {"heads": heads, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0, "v_mix": True}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff, "limit": 7.0}, "router": {"experts": experts, "top": top},
+           "shared": {"ff": expert_ff, "limit": 7.0}}
+    mlps = [{"kind": "dense", "ff": (top + 1) * expert_ff}] + [moe] * 7
+    return {"architecture": "Tatelorn", "vocab": vocab, "width": width, "max_positions": positions, "norm": {"eps": 1e-6},
+            "embedding": {"scale": width ** 0.5}, "logit_scale": 0.25,
+            "layers": [{"type": "attention", "mixer": dict(att), "mlp": copy.deepcopy(f)} for f in mlps]}
+
+
+def _nogelorn_attention_shape(width, heads, experts, top, expert_ff, vocab=32768):
+    """Nogelorn with nothing but attention layers, every key visible: rotated heads of 128 on 8 key/value heads with a sink and a gate
+    per head; the feed-forwards of the shape above with silu."""
+    att = {"heads": heads, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"dims": 128, "base": 1000000.0}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": expert_ff}}
+    mlps = [{"kind": "dense", "ff": (top + 1) * expert_ff}] + [moe] * 7
+    return {"architecture": "Nogelorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5},
+            "layers": [{"type": "attention", "mixer": copy.deepcopy(att), "mlp": copy.deepcopy(f)} for f in mlps]}
+
+
+# Tatelorn shapes with layer sizes of real models; beside each the Nogelorn shape of attention layers only, of equal width, heads,
+# layers and expert weights (its closest relative: post-norms, attention with a sink, experts chosen by the softmax over the chosen
+# with a shared one) and the Qwen3 dense shape of equal active size.
+TATELORN_SHAPES: Dict[str, dict] = {
+    "t2k-moe": _tatelorn_shape(2048, 16, 64, 5, 1408),
+    "t4k-moe": _tatelorn_shape(4096, 32, 64, 5, 2048),
+}
+NOGELORN_ATTENTION_SHAPES: Dict[str, dict] = {
+    "n2k-att": _nogelorn_attention_shape(2048, 16, 64, 5, 1408),
+    "n4k-att": _nogelorn_attention_shape(4096, 32, 64, 5, 2048),
+}
+EQUAL_NOGELORN.update({"t2k-moe": "n2k-att", "t4k-moe": "n4k-att"})
+EQUAL_QWEN3.update({"t2k-moe": _qwen3_shape(2048, 16, 8, 6 * 1408), "t4k-moe": _qwen3_shape(4096, 32, 8, 6 * 2048)})
 DESIGN_SHAPES = {"galodra": GALODRA_SHAPES, "lekilix": LEKILIX_SHAPES, "senadra": SENADRA_SHAPES, "nogelorn": NOGELORN_SHAPES,
-                 "ferodra": FERODRA_SHAPES}
+                 "ferodra": FERODRA_SHAPES, "tatelorn": TATELORN_SHAPES}
 # what each design is measured beside
 COMPARED_WITH = {"galodra": ("qwen3",), "lekilix": ("qwen3",), "senadra": ("qwen3",), "nogelorn": ("lekilix", "qwen3"),
-                 "ferodra": ("nogelorn", "qwen3")}
+                 "ferodra": ("nogelorn", "qwen3"), "tatelorn": ("nogelorn", "qwen3")}
 FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "bf16_tflops_sustained": 1400.0}
 
 
@@ -226,13 +264,19 @@ def shape_config(name: str, layers: Optional[int] = None):
         if layers:
             raw["layers"] = raw["layers"][:layers]
         return senadra_config_from_dict(raw)
-    if name in NOGELORN_SHAPES:
+    if name in NOGELORN_SHAPES or name in NOGELORN_ATTENTION_SHAPES:
         from ..models.nogelorn import nogelorn_config_from_dict
-        raw = dict(NOGELORN_SHAPES[name])
+        raw = dict(NOGELORN_SHAPES.get(name) or NOGELORN_ATTENTION_SHAPES[name])
         if layers:
             raw["layers"] = raw["layers"][:layers]
-            raw["loop"] = None if layers < raw["loop"]["stop"] else raw["loop"]
+            raw["loop"] = None if raw.get("loop") is None or layers < raw["loop"]["stop"] else raw["loop"]
         return nogelorn_config_from_dict(raw)
+    if name in TATELORN_SHAPES:
+        from ..models.tatelorn import tatelorn_config_from_dict
+        raw = dict(TATELORN_SHAPES[name])
+        if layers:
+            raw["layers"] = raw["layers"][:layers]
+        return tatelorn_config_from_dict(raw)
     if name in FERODRA_SHAPES:
         from ..models.ferodra import ferodra_config_from_dict
         raw = dict(FERODRA_SHAPES[name])
@@ -256,7 +300,8 @@ def random_model(name: str, dtype: str = "bfloat16", device="cuda:0", seed: int 
     from ..engine.model import Model
     cfg = shape_config(name, layers)
     arch = ("Galodra" if name in GALODRA_SHAPES else "Lekilix" if name in LEKILIX_SHAPES else "Senadra" if name in SENADRA_SHAPES
-            else "Nogelorn" if name in NOGELORN_SHAPES else "Ferodra" if name in FERODRA_SHAPES else "Qwen3ForCausalLM")
+            else "Nogelorn" if name in NOGELORN_SHAPES or name in NOGELORN_ATTENTION_SHAPES
+            else "Ferodra" if name in FERODRA_SHAPES else "Tatelorn" if name in TATELORN_SHAPES else "Qwen3ForCausalLM")
     model = Model.from_random(get_architecture(arch), cfg, seed=seed, dtype=dtype, device=device, norm_jitter=0.0)
     if arch == "Ferodra":
         # a norm by tanh does not bring a small stream to unit size: with rows of N(0, 0.02) every token would look alike to the
@@ -269,6 +314,8 @@ def accounting_for(cfg, dtype_bytes: int = 2):
     """Bytes and flops of a step for a configuration of any built-in architecture."""
     if type(cfg).__name__ == "FerodraConfig":
         return FerodraAccounting(cfg, dtype_bytes)
+    if type(cfg).__name__ == "TatelornConfig":
+        return TatelornAccounting(cfg, dtype_bytes)
     if type(cfg).__name__ == "NogelornConfig":
         return NogelornAccounting(cfg, dtype_bytes)
     if hasattr(cfg, "embedding_scale"):
@@ -519,6 +566,41 @@ class FerodraAccounting:
                 total += 2.0 * m.heads * 2 * (m.dim + m.vdim) * tokens * (tokens + 1) / 2
             else:
                 total += 6.0 * tokens * m.heads * m.dim * m.vdim          # S^T k, the update and the read-out of every token
+        return total
+
+
+class TatelornAccounting:
+    """Bytes and flops of a Tatelorn step.  A decode step reads every dense weight once, of the experts those that the batch is
+    expected to reach plus the shared one, and every cell of the K/V cache."""
+
+    def __init__(self, cfg, dtype_bytes: int = 2):
+        self.cfg, self.b = cfg, dtype_bytes
+        self.head_w = cfg.vocab * cfg.width
+
+    def _layer(self, lc, batch: int):
+        """(weights read by a step of ``batch`` tokens, weights a token multiplies with) of one layer."""
+        w, m, f = self.cfg.width, lc.mixer, lc.mlp
+        mix = w * (m.heads + m.kv_heads) * m.dim + w * m.kv_heads * m.vdim + m.heads * m.vdim * w
+        if f is None:
+            return mix, mix
+        if f.kind == "dense":
+            return mix + 3 * w * f.ff, mix + 3 * w * f.ff
+        reached = f.experts * (1.0 - (1.0 - f.top / f.experts) ** batch)
+        fixed = w * f.experts + (w * (1 + 3 * f.shared_ff) if f.shared_ff else 0)
+        return mix + fixed + reached * 3 * w * f.ff, mix + fixed + f.top * 3 * w * f.ff
+
+    def decode_bytes(self, batch: int, ctx_avg: float) -> float:
+        total = self.head_w * self.b
+        for lc in self.cfg.layers:
+            m = lc.mixer
+            total += self._layer(lc, batch)[0] * self.b + batch * ctx_avg * m.kv_heads * (m.dim + m.vdim) * self.b
+        return total
+
+    def prefill_flops(self, tokens: int) -> float:
+        total = 2.0 * self.head_w
+        for lc in self.cfg.layers:
+            m = lc.mixer
+            total += 2.0 * tokens * self._layer(lc, 1)[1] + 2.0 * m.heads * (m.dim + m.vdim) * tokens * (tokens + 1) / 2
         return total
 
 
