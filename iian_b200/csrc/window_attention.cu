@@ -138,16 +138,18 @@ template <int U, int R, typename A>
 __global__ void head_norm_store_kernel(const A * __restrict__ proj, long long ld, int q_off, int k_off, int v_off, A * __restrict__ q_out,
                                        A * __restrict__ k_cache, A * __restrict__ v_cache, const float * __restrict__ q_weight,
                                        const float * __restrict__ k_weight, const A * __restrict__ first, long long ld_first, float keep,
-                                       float share, const int * __restrict__ slots, long long items, int nh, int nkv, int dk, int dv,
-                                       int L, int page_size, long long n_cells, float eps) {
+                                       float share, const int * __restrict__ slots, unsigned items, int nh, int nkv, int dk, int dv,
+                                       int log_l, int page_size, int n_cells, float eps) {
     pdl_wait();
     pdl_launch_dependents();
-    const long long item = ((long long) blockIdx.x * blockDim.x + threadIdx.x) / L;
+    const int L = 1 << log_l;
+    const unsigned item = blockIdx.x * (blockDim.x >> log_l) + (threadIdx.x >> log_l);
     const int lane = threadIdx.x & (L - 1);
-    const int per_token = nh + 2 * nkv;
+    const unsigned per_token = nh + 2 * nkv;
     const bool live = item < items;                          // (every lane of a warp takes part in the sums)
-    const long long t = live ? item / per_token : 0;
-    const int hh = live ? (int) (item - t * per_token) : 0;
+    const unsigned tok = live ? item / per_token : 0;
+    const int hh = live ? (int) (item - tok * per_token) : 0;
+    const long long t = tok;
     const int kind = hh < nh ? 0 : hh < nh + nkv ? 1 : 2;    // query, key, value
     const int g = kind == 0 ? hh : kind == 1 ? hh - nh : hh - nh - nkv;
     const int n = kind == 2 ? dv : dk;
@@ -169,9 +171,10 @@ __global__ void head_norm_store_kernel(const A * __restrict__ proj, long long ld
     if (kind == 0) {
         dst = q_out + (t * nh + g) * (long long) dk;
     } else {
-        const long long cell = slots[t];
+        const int cell = slots[t];
         if (cell < 0 || cell >= n_cells) return;             // padding token: nothing is stored
-        const long long row = (cell / page_size * nkv + g) * page_size + cell % page_size;
+        const int page = cell / page_size;
+        const long long row = ((long long) page * nkv + g) * page_size + (cell - page * page_size);
         dst = kind == 1 ? k_cache + row * dk : v_cache + row * dv;
     }
     const float * w = kind == 0 ? q_weight : kind == 1 ? k_weight : nullptr;
@@ -182,8 +185,15 @@ __global__ void head_norm_store_kernel(const A * __restrict__ proj, long long ld
         const int c = (lane + r * L) * U;
         if (c >= n) continue;
         if (w != nullptr) {
+            if constexpr (U > 1) {                           // (the weights are 16-byte aligned and c a multiple of 4)
 #pragma unroll
-            for (int i = 0; i < U; i++) f[r][i] = f[r][i] * inv * w[c + i];
+                for (int i = 0; i < U; i += 4) {
+                    const float4 w4 = *reinterpret_cast<const float4 *>(w + c + i);
+                    f[r][i] *= inv * w4.x; f[r][i + 1] *= inv * w4.y; f[r][i + 2] *= inv * w4.z; f[r][i + 3] *= inv * w4.w;
+                }
+            } else {
+                f[r][0] *= inv * w[c];
+            }
         } else if (other != nullptr) {
             float o[U];
             wa_load<U>(other + c, o);
@@ -348,17 +358,19 @@ IIAN_API int iian_head_norm_store(const void * proj, long long ld, int q_off, in
     const int full = act_dtype == IIAN_F32 ? 4 : 8;
     const bool vec = dk % full == 0 && dv % full == 0 && ld % full == 0 && q_off % full == 0 && k_off % full == 0 && v_off % full == 0 &&
                      ld_first % full == 0 &&
-                     (((uintptr_t) proj | (uintptr_t) q_out | (uintptr_t) k_cache | (uintptr_t) v_cache | (uintptr_t) first) & 15) == 0;
+                     (((uintptr_t) proj | (uintptr_t) q_out | (uintptr_t) k_cache | (uintptr_t) v_cache | (uintptr_t) first |
+                       (uintptr_t) q_weight | (uintptr_t) k_weight) & 15) == 0;
     const int U = vec ? full : 1;
     const int units = ((dk > dv ? dk : dv) + U - 1) / U;
-    int L = 1;
-    while (L < units && L < 32) L *= 2;
-    const int R = (units + L - 1) / L;
+    int log_l = 0;
+    while ((1 << log_l) < units && log_l < 5) log_l++;
+    const int L = 1 << log_l, R = (units + L - 1) / L;
     const long long items = (long long) N * (nh + 2 * nkv);
+    if (items > (1LL << 30) || n_cells > 2147483647LL) return IIAN_ERR_LIMIT;
     const unsigned blocks = (unsigned) ((items * L + 255) / 256);
 #define IIAN_HNS(U, R, A) return iian_launch(head_norm_store_kernel<U, R, A>, dim3(blocks), dim3(256), 0, stream, (const A *) proj, ld, q_off, \
-        k_off, v_off, (A *) q_out, (A *) k_cache, (A *) v_cache, q_weight, k_weight, (const A *) first, ld_first, keep, share, slots, items, \
-        nh, nkv, dk, dv, L, page_size, n_cells, eps)
+        k_off, v_off, (A *) q_out, (A *) k_cache, (A *) v_cache, q_weight, k_weight, (const A *) first, ld_first, keep, share, slots, (unsigned) items, \
+        nh, nkv, dk, dv, log_l, page_size, (int) n_cells, eps)
     if (act_dtype == IIAN_F32) {
         if (vec && R == 1) IIAN_HNS(4, 1, float);
         if (vec) IIAN_HNS(4, 4, float);
